@@ -130,13 +130,26 @@ __global__ void __launch_bounds__(256) k_seq_rms(AT* out, const float* x, const 
 }
 
 // RMS norm with a weight over `len` columns of src rows: segment s of blockIdx.y.  Segment 0 goes to an activation
-// matrix, segment 1 (the cached latent) to its cache row.
+// matrix, segment 1 (the cached latent) to its cache row; behind the latent the cache row holds the key part that all heads
+// share, `rope.dims` channels of the projection turned by the token's position (not normed).
 struct RmsSeg {
 	int col, len;
 	const bf16* w;
 };
+// rotation of channels 2i and 2i + 1 by position * freq[i] (angles in double, cos and sin times `mag`)
+struct PairRope {
+	int dims;           // even; 0: none
+	const double* freq; // [dims / 2]
+	float mag;
+};
+__device__ __forceinline__ float2 rope_pair(const PairRope& r, int pos, int i, float u, float v) {
+	double sd, cd;
+	sincos((double)pos * r.freq[i], &sd, &cd);
+	const float c = (float)cd * r.mag, s = (float)sd * r.mag;
+	return make_float2(u * c - v * s, v * c + u * s);
+}
 template <typename AT>
-__global__ void k_seq_latent_norm(const float* proj, int ldp, RmsSeg sq, RmsSeg sc, AT* cq, float* cache, SeqBatch sb, float eps) {
+__global__ void k_seq_latent_norm(const float* proj, int ldp, RmsSeg sq, RmsSeg sc, AT* cq, float* cache, PairRope rope, SeqBatch sb, float eps) {
 	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
 	const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 	const int n = blockIdx.x * (blockDim.x >> 5) + warp;
@@ -151,8 +164,31 @@ __global__ void k_seq_latent_norm(const float* proj, int ldp, RmsSeg sq, RmsSeg 
 		AT* d = cq + (size_t)n * s.len;
 		for (int i = lane; i < s.len; i += 32) d[i] = to_act<AT>(src[i] * r * ldf(s.w + i));
 	} else {
-		float* d = cache + cache_row(sb, sb.tslot[n], sb.tpos[n]) * s.len;
+		const int pos = sb.tpos[n];
+		float* d = cache + cache_row(sb, sb.tslot[n], pos) * (s.len + rope.dims);
 		for (int i = lane; i < s.len; i += 32) d[i] = src[i] * r * ldf(s.w + i);
+		for (int i = lane; i < rope.dims / 2; i += 32) {
+			const float2 t = rope_pair(rope, pos, i, src[s.len + 2 * i], src[s.len + 2 * i + 1]);
+			d[s.len + 2 * i] = t.x, d[s.len + 2 * i + 1] = t.y;
+		}
+	}
+}
+// the rotated query channels of every head: q[n][h * ldh + col + d] from src [N][heads * dims]; one CTA per token, the angles are formed once
+__global__ void __launch_bounds__(128) k_seq_rope_heads(float* q, const float* src, int heads, long ldq, int ldh, int col, PairRope rope, SeqBatch sb) {
+	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
+	extern __shared__ float2 cs2[]; // [dims / 2] (cos, sin)
+	const int n = blockIdx.x, half = rope.dims / 2;
+	for (int i = threadIdx.x; i < half; i += blockDim.x) {
+		double s, c;
+		sincos((double)sb.tpos[n] * rope.freq[i], &s, &c);
+		cs2[i] = make_float2((float)c * rope.mag, (float)s * rope.mag);
+	}
+	__syncthreads();
+	for (int e = threadIdx.x; e < heads * half; e += blockDim.x) {
+		const int h = e / half, i = e % half;
+		const float u = src[(size_t)n * heads * rope.dims + 2 * e], v = src[(size_t)n * heads * rope.dims + 2 * e + 1];
+		float* d = q + (size_t)n * ldq + (size_t)h * ldh + col + 2 * i;
+		d[0] = u * cs2[i].x - v * cs2[i].y, d[1] = v * cs2[i].x + u * cs2[i].y;
 	}
 }
 
@@ -298,7 +334,7 @@ __global__ void k_seq_conv_state(float* state, const float* proj, int ldp, int t
 #define ATT_KC 64
 #define ATT_THREADS 256
 #define ATT_MAXI 32 // output elements per thread: heads of the tile x value columns per thread
-#define ATT_KPL 16  // key channels per lane held in registers (keys up to 512 wide)
+#define ATT_KPL 18  // key channels per lane held in registers (keys up to 576 wide: a 512-wide latent with its 64 rotated channels)
 struct AttArgs {
 	const float* q;   // [N][heads][kd]
 	const float* kc;  // cache rows of width kld
@@ -1505,6 +1541,128 @@ __global__ void __launch_bounds__(256) k_seq_post_norm(float* x, AT* act, const 
 	}
 	for (int c = (PN_KEEP * nt + tid) * V; c < width; c += nt * V) put(c, yval(c));
 }
+// Sandwich blocks: what follows a sublayer's last product, in one pass over the row.
+//   y = (base + the routed experts' sum) * sigmoid(gate),  v = x[n] + y / sqrt(mean(y^2) + eps) * (w + offset);
+//   with a depth average (dwa): X_k = v is kept in hist[k] and v becomes dwa[k] v + sum_(j < k) dwa[j] hist[j];
+//   x[n] = v;  act[n] = v / sqrt(mean(v^2) + eps) * (w_next + offset), the normed input of the sublayer that follows (w_next null: none).
+// One CTA per token; V and PN_KEEP as in k_seq_post_norm.
+struct Sandwich {
+	const float* base; // a sublayer's last product, or null
+	HcMoe moe;
+	const float* gate; // gate[n * ldg + c], raw; null: none
+	long ldg;
+	const bf16* w;
+	float* hist;       // [k + 1 ..][N][width]
+	const bf16* dwa;   // [k + 1], or null
+	int k;
+	const bf16* w_next;
+	float offset, eps;
+};
+template <typename AT, int V>
+__global__ void __launch_bounds__(256) k_seq_sandwich(float* x, AT* act, Sandwich a, int N, int width) {
+	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
+	__shared__ float red[2][8];
+	const int tid = threadIdx.x, nt = blockDim.x;
+	const size_t n = blockIdx.x;
+	auto yval = [&](int c) {
+		HcVec<V> y;
+#pragma unroll
+		for (int e = 0; e < V; ++e) y.v[e] = 0.f;
+		if (a.base) y = hc_load<V>(a.base + n * width + c);
+		if (a.moe.y)
+			for (int k = 0; k < a.moe.top; ++k) {
+				const HcVec<V> v = hc_load<V>(a.moe.y + (size_t)a.moe.inv[n * a.moe.top + k] * width + c);
+				const float wk = a.moe.wt ? a.moe.wt[n * a.moe.top + k] : 1.f;
+#pragma unroll
+				for (int e = 0; e < V; ++e) y.v[e] = a.moe.wt ? fmaf(wk, v.v[e], y.v[e]) : y.v[e] + v.v[e];
+			}
+		if (a.gate) {
+			const HcVec<V> g = hc_load<V>(a.gate + n * a.ldg + c);
+#pragma unroll
+			for (int e = 0; e < V; ++e) y.v[e] *= sigmoidf_(g.v[e]);
+		}
+		return y;
+	};
+	auto row_sum = [&](float ss, float* r) { // every thread adds the warps' sums in the same order
+		ss = warp_sum(ss);
+		if ((tid & 31) == 0) r[tid >> 5] = ss;
+		__syncthreads();
+		ss = 0.f;
+		for (int i = 0; i < (nt >> 5); ++i) ss += r[i];
+		return ss;
+	};
+	HcVec<V> keep[PN_KEEP];
+	float ss = 0.f;
+#pragma unroll
+	for (int i = 0; i < PN_KEEP; ++i) {
+		const int c = (i * nt + tid) * V;
+		if (c < width) keep[i] = yval(c);
+		else {
+#pragma unroll
+			for (int e = 0; e < V; ++e) keep[i].v[e] = 0.f;
+		}
+#pragma unroll
+		for (int e = 0; e < V; ++e) ss = fmaf(keep[i].v[e], keep[i].v[e], ss);
+	}
+	for (int c = (PN_KEEP * nt + tid) * V; c < width; c += nt * V) {
+		const HcVec<V> y = yval(c);
+#pragma unroll
+		for (int e = 0; e < V; ++e) ss = fmaf(y.v[e], y.v[e], ss);
+	}
+	const float rinv = 1.f / sqrtf(row_sum(ss, red[0]) / (float)width + a.eps);
+	float* xr = x + n * width;
+	auto put = [&](int c, const HcVec<V>& y) { // the new row's columns c .. c + V - 1
+		HcVec<V> v = hc_load<V>(xr + c);
+#pragma unroll
+		for (int e = 0; e < V; ++e) v.v[e] += y.v[e] * rinv * (ldf(a.w + c + e) + a.offset);
+		if (a.dwa) {
+			const size_t o = n * width + c, layer = (size_t)N * width;
+			hc_store<V>(a.hist + a.k * layer + o, v);
+			HcVec<V> m;
+#pragma unroll
+			for (int e = 0; e < V; ++e) m.v[e] = 0.f;
+#pragma unroll 4
+			for (int j = 0; j < a.k; ++j) {
+				const HcVec<V> h = hc_load<V>(a.hist + j * layer + o);
+				const float wj = ldf(a.dwa + j);
+#pragma unroll
+				for (int e = 0; e < V; ++e) m.v[e] = fmaf(wj, h.v[e], m.v[e]);
+			}
+			const float wk = ldf(a.dwa + a.k);
+#pragma unroll
+			for (int e = 0; e < V; ++e) v.v[e] = fmaf(wk, v.v[e], m.v[e]);
+		}
+		hc_store<V>(xr + c, v);
+		return v;
+	};
+	ss = 0.f;
+#pragma unroll
+	for (int i = 0; i < PN_KEEP; ++i) {
+		const int c = (i * nt + tid) * V;
+		if (c < width) keep[i] = put(c, keep[i]);
+#pragma unroll
+		for (int e = 0; e < V; ++e) ss = fmaf(keep[i].v[e], keep[i].v[e], ss); // columns past the row are still zero
+	}
+	for (int c = (PN_KEEP * nt + tid) * V; c < width; c += nt * V) {
+		const HcVec<V> v = put(c, yval(c));
+#pragma unroll
+		for (int e = 0; e < V; ++e) ss = fmaf(v.v[e], v.v[e], ss);
+	}
+	if (!a.w_next) return;
+	const float rnext = 1.f / sqrtf(row_sum(ss, red[1]) / (float)width + a.eps);
+	AT* ar = act + n * width;
+	auto normed = [&](int c, HcVec<V> v) {
+#pragma unroll
+		for (int e = 0; e < V; ++e) v.v[e] *= rnext * (ldf(a.w_next + c + e) + a.offset);
+		pn_store_act<AT, V>(ar + c, v);
+	};
+#pragma unroll
+	for (int i = 0; i < PN_KEEP; ++i) {
+		const int c = (i * nt + tid) * V;
+		if (c < width) normed(c, keep[i]);
+	}
+	for (int c = (PN_KEEP * nt + tid) * V; c < width; c += nt * V) normed(c, hc_load<V>(xr + c)); // written by this very thread
+}
 // out[n] = sum of the streams of token n
 __global__ void k_seq_stream_sum(float* out, const float* x, int N, int width, int streams) {
 	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
@@ -1682,6 +1840,86 @@ __global__ void k_seq_lin_out(AT* out, LinOut a, int N) {
 		if (a.gate_mode == 1) v *= sigmoidf_(a.gate[n * a.ldg + c]);
 		out[n * inner + c] = to_act<AT>(v);
 	}
+}
+
+// ---------------------------------------------------------------- gated recurrence whose gates read only the current token (minGRU)
+// Per channel  S <- (1 - z) S + z c,  z = sigmoid(raw z),  c = u + 1/2 (u >= 0) or sigmoid(u) (u < 0);  output S silu(g).  Raw z, u and g are
+// columns 0, width and 2 width of the projection.  The map of a stretch of tokens on the state is S -> A S + B, so a prompt is cut into
+// chunks of `chunk` tokens: k_seq_mingru_chunk forms every chunk's (A, B) but the last's, k_seq_mingru_apply folds those before its chunk
+// into the state its chunk starts from and runs the tokens.  A sequence of at most `chunk` new tokens (a decoded one) needs the second kernel only.
+struct MinGruArgs {
+	const float* proj;
+	int ldp, width;
+	float* state;  // [slots][width]
+	float2* carry; // [B][slots of carry][width]: entry 0 = (0, state before the step), entry k + 1 = (A, B) of chunk k
+	int chunk, carries;
+};
+__device__ __forceinline__ void mingru_step(float zr, float u, float& keep, float& take) { // S <- keep S + take
+	const float z = sigmoidf_(zr);
+	keep = 1.f - z, take = z * (u >= 0.f ? u + 0.5f : sigmoidf_(u));
+}
+#define MINGRU_U 8 // tokens whose inputs are requested together
+__global__ void __launch_bounds__(64) k_seq_mingru_chunk(MinGruArgs a, SeqBatch sb) {
+	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
+	const int ch = blockIdx.x * 64 + threadIdx.x, k = blockIdx.y, b = blockIdx.z, cnt = sb.scount[b];
+	if (ch >= a.width || (long)(k + 1) * a.chunk >= cnt) return; // the last chunk's map is not needed
+	float2* cr = a.carry + (size_t)b * a.carries * a.width + ch;
+	if (k == 0) cr[0] = make_float2(0.f, a.state[(size_t)sb.sslot[b] * a.width + ch]);
+	const float* p = a.proj + (size_t)(sb.sstart[b] + k * a.chunk) * a.ldp + ch;
+	float A = 1.f, B = 0.f;
+	for (int t0 = 0; t0 < a.chunk; t0 += MINGRU_U) {
+		float zr[MINGRU_U], u[MINGRU_U];
+#pragma unroll
+		for (int i = 0; i < MINGRU_U; ++i)
+			if (t0 + i < a.chunk) zr[i] = p[(size_t)(t0 + i) * a.ldp], u[i] = p[(size_t)(t0 + i) * a.ldp + a.width];
+#pragma unroll
+		for (int i = 0; i < MINGRU_U; ++i)
+			if (t0 + i < a.chunk) {
+				float keep, take;
+				mingru_step(zr[i], u[i], keep, take);
+				A *= keep, B = fmaf(keep, B, take);
+			}
+	}
+	cr[(size_t)(k + 1) * a.width] = make_float2(A, B);
+}
+template <typename AT>
+__global__ void __launch_bounds__(64) k_seq_mingru_apply(MinGruArgs a, AT* out, SeqBatch sb) {
+	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
+	const int ch = blockIdx.x * 64 + threadIdx.x, k = blockIdx.y, b = blockIdx.z, cnt = sb.scount[b];
+	if (ch >= a.width || (long)k * a.chunk >= cnt) return;
+	float* st = a.state + (size_t)sb.sslot[b] * a.width + ch;
+	float S;
+	if (cnt <= a.chunk) S = *st;
+	else { // the state itself is written below by the last chunk while others still start: all of them read entry 0 instead
+		S = 0.f;
+		const float2* cr = a.carry + (size_t)b * a.carries * a.width + ch;
+#pragma unroll 8
+		for (int j = 0; j <= k; ++j) {
+			const float2 m = cr[(size_t)j * a.width];
+			S = fmaf(m.x, S, m.y);
+		}
+	}
+	const int first = sb.sstart[b] + k * a.chunk, nt = min(a.chunk, cnt - k * a.chunk);
+	const float* p = a.proj + (size_t)first * a.ldp + ch;
+	AT* o = out + (size_t)first * a.width + ch;
+	for (int t0 = 0; t0 < nt; t0 += MINGRU_U) {
+		float zr[MINGRU_U], u[MINGRU_U], g[MINGRU_U];
+#pragma unroll
+		for (int i = 0; i < MINGRU_U; ++i)
+			if (t0 + i < nt) {
+				const float* q = p + (size_t)(t0 + i) * a.ldp;
+				zr[i] = q[0], u[i] = q[a.width], g[i] = q[2 * a.width];
+			}
+#pragma unroll
+		for (int i = 0; i < MINGRU_U; ++i)
+			if (t0 + i < nt) {
+				float keep, take;
+				mingru_step(zr[i], u[i], keep, take);
+				S = fmaf(keep, S, take);
+				o[(size_t)(t0 + i) * a.width] = to_act<AT>(S * g[i] * sigmoidf_(g[i]));
+			}
+	}
+	if (k * a.chunk + nt == cnt) *st = S;
 }
 
 // ---------------------------------------------------------------- products  Y[n][m] = sum_k X[n][k] W[m][k]

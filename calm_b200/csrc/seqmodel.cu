@@ -21,18 +21,19 @@ namespace {
 
 uint64_t g_seq_launches = 0;
 
-enum Kind { KD_EMBED, KD_NORM, KD_GEMM, KD_GEMM_TC, KD_GEMM_SKINNY, KD_CONV, KD_ATTN_LATENT, KD_ATTN_WINDOW, KD_DELTA, KD_ELEMENT, KD_QK, KD_GLA, KD_ROUTE, KD_HYPER, KD_LINPREP, KD_COUNT };
+enum Kind { KD_EMBED, KD_NORM, KD_GEMM, KD_GEMM_TC, KD_GEMM_SKINNY, KD_CONV, KD_ATTN_LATENT, KD_ATTN_WINDOW, KD_DELTA, KD_ELEMENT, KD_QK, KD_GLA, KD_ROUTE, KD_HYPER, KD_LINPREP, KD_MINGRU, KD_COUNT };
 const char* const kKindNames[KD_COUNT] = {"embed", "norm", "gemm", "gemm_tcgen05", "gemm_skinny", "conv", "attention_latent", "attention_window", "delta_scan", "elementwise",
-                                          "qk_prep", "gla_scan", "moe_route", "hyper", "lin_prep"};
+                                          "qk_prep", "gla_scan", "moe_route", "hyper", "lin_prep", "mingru_scan"};
 
 // what one run of a layer owns (a looped layer has one of these per pass)
 struct RunState {
 	int layer = 0;
 	bool readd = false;      // the embedding output is added to the stream right before this run
-	float* cache_a = nullptr; // SEQ_LATENT: latent rows; SEQ_WINDOW / SEQ_GQA: key rows
+	float* cache_a = nullptr; // SEQ_LATENT: latent rows (with the shared rotated key part behind each; an earlier layer's with kv_shared); SEQ_WINDOW / SEQ_GQA: key rows
 	float* cache_b = nullptr; // SEQ_WINDOW / SEQ_GQA: value rows
 	float* conv = nullptr;    // [slots][taps-1][channels]
-	float* delta = nullptr;   // SEQ_DELTA / SEQ_GLA: the recurrent state [slots][heads][dim][vdim]
+	bool cache_borrowed = false; // SEQ_LATENT with kv_shared: cache_a belongs to another run
+	float* delta = nullptr;   // SEQ_DELTA / SEQ_GLA: the recurrent state [slots][heads][dim][vdim]; SEQ_MINGRU: [slots][dim]
 	size_t conv_per_slot = 0, delta_per_slot = 0;
 	float* mstate = nullptr;  // SEQ_MLSTM: the running maximum of the log gates [slots][heads]
 	size_t m_per_slot = 0;
@@ -52,7 +53,7 @@ struct Seq {
 	std::vector<SeqLayer> layers;
 	std::vector<std::array<SeqLayer, 2>> pairs;
 	std::vector<RunState> runs;
-	std::map<const SeqLayer*, std::pair<double*, float>> rot; // per SEQ_GQA record (a layer's, or one of a pair's): angle step of every rotated pair (device), factor on cos and sin
+	std::map<const SeqLayer*, std::pair<double*, float>> rot; // per SEQ_GQA / SEQ_LATENT record (a layer's, or one of a pair's): angle step of every rotated pair (device), factor on cos and sin
 	cudaStream_t stream = nullptr;
 	int sms = 0;
 	bool tc = false; // tcgen05 products available (bf16 mode)
@@ -72,6 +73,10 @@ struct Seq {
 
 	// workspace for cap_tokens tokens
 	float *x = nullptr, *x0 = nullptr, *proj = nullptr, *f[6] = {};
+	float* hist = nullptr;                            // depth average: X_0 (the embedding rows), X_1 .. X_layers of the step's tokens, [layers + 1][N][width]
+	bool depth = false;                               // some layer averages over depth
+	float2* carry = nullptr;                          // SEQ_MINGRU: chunk maps of a step's longer portions
+	size_t carry_cap = 0;
 	void* ah = nullptr;                               // parallel blocks: a dense unit's hidden activations, written by the mixer's input product
 	size_t w_ah = 0;
 	float* mo = nullptr;                              // parallel blocks: the mixer's output until the feed-forward's is added with it; hyper blocks: a sublayer's output
@@ -158,7 +163,8 @@ void launch_k(Seq& s, void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t sm
 
 size_t in_rows(const SeqLayer& L) {
 	switch (L.type) {
-	case SEQ_LATENT: return (size_t)L.q_rank + L.kv_rank + L.heads;
+	case SEQ_LATENT: return (size_t)L.q_rank + (L.kv_shared ? 0 : L.kv_rank + L.rot_dims) + (L.no_gate ? 0 : L.heads);
+	case SEQ_MINGRU: return (size_t)3 * L.dim;
 	case SEQ_DELTA: return (size_t)2 * L.kv_heads * L.dim + (size_t)L.heads * L.vdim + L.heads + L.a_rank + L.g_rank;
 	case SEQ_GQA: return (size_t)L.heads * L.dim + (size_t)L.kv_heads * L.dim + (size_t)L.kv_heads * L.vdim + (L.no_gate ? 0 : L.gate_per_head ? (size_t)L.heads : (size_t)L.heads * L.vdim);
 	case SEQ_MLSTM: return (size_t)2 * L.heads * L.dim + (size_t)2 * L.heads * L.vdim + 2 * L.heads;
@@ -181,6 +187,10 @@ int pair_stride(const SeqLayer& L) {
 	const size_t m = pair_offset(L) + in_rows(L.pair[1]) - (L.pair[1].type == SEQ_GLA ? L.pair[1].a_rank : 0);
 	return (int)((m + 3) & ~(size_t)3);
 }
+// sandwich blocks with a residual gate: the gate's `width` rows lead the sublayer's first matrix, whose fp32 product is gate_cols + rows wide
+int gate_cols(const SeqModel& m) { return m.block == SEQ_BLOCK_SANDWICH && m.res_gate ? m.width : 0; }
+int gated_stride(const SeqModel& m, size_t rows) { return (int)((gate_cols(m) + rows + 3) & ~(size_t)3); }
+int mixer_stride(const SeqModel& m, const SeqLayer& L) { return gate_cols(m) ? gated_stride(m, in_rows(L)) : proj_stride(L); }
 int conv_channels(const SeqLayer& L) {
 	if (L.type == SEQ_DELTA) return 2 * L.kv_heads * L.dim + L.heads * L.vdim;
 	if (L.type == SEQ_WINDOW) return L.heads * L.dim + L.kv_heads * L.dim + L.kv_heads * L.vdim;
@@ -247,7 +257,17 @@ void validate_mixer(const Seq& s, int i, const SeqLayer& L, bool inner) {
 			}
 		} else if (L.type == SEQ_LATENT) {
 			if (L.q_rank < 1 || L.kv_rank < 1) CALM_FATAL("seq: layer %d: latent ranks must be positive", i);
-			if (cdiv(L.kv_rank, ATT_THREADS) > ATT_MAXI) CALM_FATAL("seq: layer %d: kv_rank %d is more than the attention kernel holds", i, L.kv_rank);
+			if (L.rot_dims < 0 || L.rot_dims % 2) CALM_FATAL("seq: layer %d: rot_dims must be even", i);
+				if (L.rot_dims > 0 && !(L.rot_base > 0.f)) CALM_FATAL("seq: layer %d: rot_base must be positive", i);
+				if (L.kv_shared) {
+					const int j = L.kv_shared - 1;
+					if (inner || j < 0 || j >= i) CALM_FATAL("seq: layer %d: kv_shared names an earlier layer", i);
+					const SeqLayer& o = s.layers[j];
+					if (o.type != SEQ_LATENT || o.kv_shared || o.kv_rank != L.kv_rank || o.rot_dims != L.rot_dims || o.rot_base != L.rot_base || o.rot_factor != L.rot_factor)
+						CALM_FATAL("seq: layer %d: kv_shared needs a latent attention with its own latent of the same kv_rank and rotation", i);
+					if (m.loop_times > 1) CALM_FATAL("seq: layer %d: kv_shared is not served beside a looped span", i);
+				}
+				if (cdiv(L.kv_rank, ATT_THREADS) > ATT_MAXI) CALM_FATAL("seq: layer %d: kv_rank %d is more than the attention kernel holds", i, L.kv_rank);
 		} else if (L.type == SEQ_DELTA || L.type == SEQ_WINDOW) {
 			if (L.kv_heads < 1 || L.heads % L.kv_heads) CALM_FATAL("seq: layer %d: heads must be a multiple of kv_heads", i);
 			if (L.taps < 1) CALM_FATAL("seq: layer %d: taps must be positive", i);
@@ -267,9 +287,13 @@ void validate_mixer(const Seq& s, int i, const SeqLayer& L, bool inner) {
 			if (L.dim > 256) CALM_FATAL("seq: layer %d: a gated-linear-attention head holds at most 256 key channels", i);
 			if (L.a_rank < 1) CALM_FATAL("seq: layer %d: the decay rank must be positive", i);
 			if (!(L.tau > 0.f)) CALM_FATAL("seq: layer %d: tau must be positive", i);
+		} else if (L.type == SEQ_MINGRU) {
+			if (L.heads != 1 || L.vdim != L.dim) CALM_FATAL("seq: layer %d: this recurrence is per channel: heads 1, vdim = dim", i);
 		} else CALM_FATAL("seq: layer %d: unknown mixer %d", i, L.type);
-		if ((L.type != SEQ_GQA && (L.chunk || L.dist_bias || L.add_one || L.v_norm || L.no_gate || L.qk_per_head || L.gate_per_head || L.scores_f32)) || L.chunk < 0)
-			CALM_FATAL("seq: layer %d: chunk, dist_bias, add_one, v_norm, no_gate, qk_per_head, gate_per_head and scores_f32 are options of SEQ_GQA", i);
+		if ((L.type != SEQ_GQA && (L.chunk || L.dist_bias || L.add_one || L.v_norm || L.qk_per_head || L.gate_per_head)) || L.chunk < 0)
+			CALM_FATAL("seq: layer %d: chunk, dist_bias, add_one, v_norm, qk_per_head and gate_per_head are options of SEQ_GQA", i);
+		if (L.type != SEQ_GQA && L.type != SEQ_LATENT && (L.no_gate || L.scores_f32)) CALM_FATAL("seq: layer %d: no_gate and scores_f32 are options of SEQ_GQA and SEQ_LATENT", i);
+		if (L.type != SEQ_LATENT && L.kv_shared) CALM_FATAL("seq: layer %d: kv_shared is an option of SEQ_LATENT", i);
 		(void)m;
 	}
 }
@@ -288,7 +312,12 @@ void validate(const Seq& s) {
 		validate_mixer(s, i, L, false);
 		if (m.block == SEQ_BLOCK_HYPER && (!L.hc1.in || !L.hc1.out || !L.hc1.mix || (L.ff > 0 && (!L.hc2.in || !L.hc2.out || !L.hc2.mix))))
 			CALM_FATAL("seq: layer %d: hyper blocks need in, out and mix of every sublayer", i);
-		if (m.block != SEQ_BLOCK_HYPER && m.block != SEQ_BLOCK_POST && (L.type == SEQ_PAIR || is_lin(L))) CALM_FATAL("seq: layer %d: this mixer is served in hyper and post-norm blocks", i);
+		const bool sandwich = m.block == SEQ_BLOCK_SANDWICH;
+		if (m.block != SEQ_BLOCK_HYPER && m.block != SEQ_BLOCK_POST && !sandwich && (L.type == SEQ_PAIR || is_lin(L))) CALM_FATAL("seq: layer %d: this mixer is served in hyper, post-norm and sandwich blocks", i);
+		if (sandwich && L.type == SEQ_PAIR && m.res_gate) CALM_FATAL("seq: layer %d: a pair has no residual gate", i);
+		if (!sandwich && (L.dwa || m.res_gate)) CALM_FATAL("seq: layer %d: depth average and residual gate are served in sandwich blocks", i);
+		if (sandwich && (!L.norm1.w || !L.norm1b.w || (L.ff > 0 && (!L.norm2.w || !L.norm2b.w)))) CALM_FATAL("seq: layer %d: sandwich blocks have a norm before and after every sublayer", i);
+		if (sandwich && m.res_gate && L.ff > 0 && (L.ff_kind == SEQ_FF_MOE) == (L.w_rg2 != nullptr)) CALM_FATAL("seq: layer %d: the feed-forward's residual gate rides with the router's rows, or is w_rg2", i);
 		if (L.ff > 0) {
 			if (L.ff_kind < SEQ_FF_CLAMPED || L.ff_kind > SEQ_FF_GATED) CALM_FATAL("seq: layer %d: unknown feed-forward kind %d", i, L.ff_kind);
 			if (L.ff_kind == SEQ_FF_GATED && L.ff_act != SEQ_ACT_SILU && L.ff_act != SEQ_ACT_GELU_TANH) CALM_FATAL("seq: layer %d: unknown activation %d", i, L.ff_act);
@@ -299,19 +328,22 @@ void validate(const Seq& s) {
 				if (m.block == SEQ_BLOCK_SERIAL) CALM_FATAL("seq: layer %d: routed experts are not served in serial blocks", i);
 				if (L.ident < 0 || L.top > L.experts + L.ident || L.shared_ff < 0) CALM_FATAL("seq: layer %d: bad identity experts or shared unit", i);
 				if (!L.w_router && L.in_tail == 0 && L.shared_ff == 0) CALM_FATAL("seq: layer %d: the router's rows ride either behind the shared unit's or in w_router", i);
-				if (m.block != SEQ_BLOCK_HYPER && (L.ident || L.route_mode == 1)) CALM_FATAL("seq: layer %d: identity experts and route_mode 1 are served in hyper blocks", i);
+				if (m.block != SEQ_BLOCK_HYPER && (L.ident || (L.route_mode == 1 && !sandwich))) CALM_FATAL("seq: layer %d: identity experts are served in hyper blocks, route_mode 1 in hyper and sandwich blocks", i);
+				if (sandwich && (L.shared_ff || !L.w_router)) CALM_FATAL("seq: layer %d: sandwich blocks serve routed experts with w_router and without a shared unit", i);
+				if (L.expert_act < 0 || L.expert_act > 2 || (L.expert_act == 2 && !sandwich)) CALM_FATAL("seq: layer %d: clamped experts are served in sandwich blocks", i);
 				if (m.block != SEQ_BLOCK_HYPER && m.block != SEQ_BLOCK_POST && L.shared_ff) CALM_FATAL("seq: layer %d: the shared unit is served in hyper and post-norm blocks", i);
 				if (L.route_mode < 0 || L.route_mode > 2) CALM_FATAL("seq: layer %d: unknown route_mode %d", i, L.route_mode);
-				if (m.block != SEQ_BLOCK_POST && (L.expert_act || L.weight_input || L.shared_gate)) CALM_FATAL("seq: layer %d: relu^2 experts, weights on the input and the gated shared unit are served in post-norm blocks", i);
-				if (m.block == SEQ_BLOCK_POST && L.shared_ff && !L.expert_act) CALM_FATAL("seq: layer %d: post-norm blocks serve the shared unit in the relu^2 form", i);
-				if (L.weight_input && !L.expert_act) CALM_FATAL("seq: layer %d: a weight on the input is served for relu^2 experts", i);
+				if (m.block != SEQ_BLOCK_POST && (L.expert_act == 1 || L.weight_input || L.shared_gate)) CALM_FATAL("seq: layer %d: relu^2 experts, weights on the input and the gated shared unit are served in post-norm blocks", i);
+				if (m.block == SEQ_BLOCK_POST && L.shared_ff && L.expert_act != 1) CALM_FATAL("seq: layer %d: post-norm blocks serve the shared unit in the relu^2 form", i);
+				if (L.weight_input && L.expert_act != 1) CALM_FATAL("seq: layer %d: a weight on the input is served for relu^2 experts", i);
 				if (L.shared_gate && !L.shared_ff) CALM_FATAL("seq: layer %d: a shared gate needs a shared unit", i);
 			}
 		}
 	}
 	if (m.norm_kind != SEQ_NORM_DYT && m.norm_kind != SEQ_NORM_RMS) CALM_FATAL("seq: unknown norm kind %d", m.norm_kind);
-	if (m.block < SEQ_BLOCK_SERIAL || m.block > SEQ_BLOCK_POST) CALM_FATAL("seq: unknown block form %d", m.block);
+	if (m.block < SEQ_BLOCK_SERIAL || m.block > SEQ_BLOCK_SANDWICH) CALM_FATAL("seq: unknown block form %d", m.block);
 	if (m.block == SEQ_BLOCK_POST && (m.norm_kind != SEQ_NORM_RMS || m.norm_scalar || m.loop_times > 1)) CALM_FATAL("seq: post-norm blocks use the RMS norm with a weight per column, outside looped spans");
+	if (m.block == SEQ_BLOCK_SANDWICH && (m.norm_kind != SEQ_NORM_RMS || m.norm_scalar || m.loop_times > 1)) CALM_FATAL("seq: sandwich blocks use the RMS norm with a weight per column, outside looped spans");
 	if (m.bigram && (m.bigram_buckets < 1 || m.bigram_mul_prev < 0 || m.bigram_mul_cur < 0)) CALM_FATAL("seq: a bigram table needs buckets >= 1 and multipliers >= 0");
 	if (m.block == SEQ_BLOCK_HYPER && m.norm_kind != SEQ_NORM_RMS) CALM_FATAL("seq: hyper blocks use the RMS norm");
 	if (m.block == SEQ_BLOCK_SERIAL && m.norm_kind != SEQ_NORM_DYT)
@@ -364,6 +396,7 @@ void reserve_tokens(Seq& s, int N, int B, int W) {
 		}
 		s.x = (float*)dalloc(cn * s.streams * s.m.width * sizeof(float));
 		s.x0 = (float*)dalloc(cn * s.m.width * sizeof(float));
+		if (s.depth) cudaFree(s.hist), s.hist = (float*)dalloc((s.layers.size() + 1) * cn * s.m.width * sizeof(float));
 		s.proj = (float*)dalloc(cn * s.w_proj * sizeof(float));
 		for (float*& p : s.f) p = (float*)dalloc(cn * s.w_f * sizeof(float));
 		s.hA = dalloc(cn * s.m.width * act_size(s));
@@ -465,7 +498,6 @@ void dyt(Seq& s, void* out, const float* x, const int* rows, const SeqNorm& nm, 
 
 // most keys a query of this attention sees (0: all earlier positions)
 int attn_span(const SeqLayer& L) {
-	if (L.type == SEQ_LATENT) return 0;
 	int span = L.window > 0 ? L.window + (L.type == SEQ_GQA ? L.keep_first : 0) : 0;
 	if (L.type == SEQ_GQA && L.chunk > 0) span = span > 0 ? std::min(span, L.chunk) : L.chunk;
 	return span;
@@ -483,6 +515,12 @@ void hc_read(Seq& s, void* out, const int* rows, const void* in, const SeqNorm& 
 int attn_nsplit(const Seq& s, int live_tokens, int tiles, int window, int longest) {
 	const int ctas = live_tokens * tiles, chunks = cdiv(window > 0 ? std::min(longest, window) : longest, ATT_KC);
 	return ctas >= 2 * s.sms ? 1 : std::max(1, std::min({chunks, 2 * s.sms / ctas, 128}));
+}
+void ensure_carry(Seq& s, size_t need) {
+	if (need <= s.carry_cap) return;
+	CUDA_CHECK(cudaStreamSynchronize(s.stream));
+	cudaFree(s.carry); // decode graphs (one token per sequence) never read it
+	s.carry = (float2*)dalloc(need * sizeof(float2)), s.carry_cap = need;
 }
 void ensure_part(Seq& s, size_t need) {
 	if (need <= s.part_cap) return;
@@ -584,14 +622,14 @@ void attention(Seq& s, int kind, AttArgs a, void* out, const SeqBatch& sb, doubl
 		});
 }
 
-void conv(Seq& s, const SeqLayer& L, RunState& r, ConvArgs& ca, const SeqBatch& sb) {
+void conv(Seq& s, const SeqLayer& L, RunState& r, ConvArgs& ca, const SeqBatch& sb, const float* proj, int ldp) {
 	const int units = ca.seg[0].heads + ca.seg[1].heads + ca.seg[2].heads;
-	ca.proj = s.proj, ca.ldp = proj_stride(L), ca.w = (const bf16*)L.conv, ca.taps = L.taps, ca.channels = conv_channels(L), ca.state = r.conv, ca.eps = s.m.eps;
+	ca.proj = proj, ca.ldp = ldp, ca.w = (const bf16*)L.conv, ca.taps = L.taps, ca.channels = conv_channels(L), ca.state = r.conv, ca.eps = s.m.eps;
 	ca.bias = (const bf16*)L.conv_b, ca.pcol = L.type == SEQ_MAMBA2 ? L.heads * L.vdim : 0; // Mamba-2: the channels start behind z
 	const double bytes = (double)sb.N * ca.channels * 8;
 	run_kernel(s, KD_CONV, bytes, 0, [&] { launch_k(s, k_seq_conv_heads, dim3(sb.N, cdiv(units, 4)), 128, 0, ca, sb); });
 	if (L.taps > 1)
-		run_kernel(s, KD_CONV, 0, 0, [&] { launch_k(s, k_seq_conv_state, dim3(cdiv(ca.channels, 128), sb.B), 128, 0, r.conv, s.proj, ca.ldp, L.taps, ca.channels, sb, ca.pcol); });
+		run_kernel(s, KD_CONV, 0, 0, [&] { launch_k(s, k_seq_conv_state, dim3(cdiv(ca.channels, 128), sb.B), 128, 0, r.conv, proj, ca.ldp, L.taps, ca.channels, sb, ca.pcol); });
 }
 
 // how a sublayer's last product lands in the stream: serial blocks apply the Dynamic Tanh norm after the sublayer and add
@@ -607,7 +645,18 @@ struct OutEpi {
 	const void* next_in = nullptr;      // ... and in the same kernel reads them for the sublayer that follows: its `in` weights and its norm
 	const SeqNorm* next_norm = nullptr;
 	const SeqNorm* post = nullptr;      // post-norm blocks: the norm the routed feed-forward's sum goes through on its way into the stream
+	const Sandwich* sand = nullptr;     // sandwich blocks: how the routed feed-forward's sum goes into the stream (its routed part is filled in there)
 };
+// sandwich blocks: gate, second norm and residual sum of a sublayer, the depth average after a layer's last one, and the next sublayer's normed input (hA)
+template <typename AT>
+void sandwich(Seq& s, const Sandwich& a, int N) {
+	const int W = s.m.width;
+	const double rows = 2.0 + (a.base ? 1 : 0) + (a.moe.y ? a.moe.top : 0) + (a.gate ? 1 : 0) + (a.dwa ? a.k + 1 : 0);
+	run_kernel(s, KD_NORM, (double)N * W * (4.0 * rows + (a.w_next ? act_size(s) : 0)), 0, [&] {
+		if (W % 4 == 0) launch_k(s, k_seq_sandwich<AT, 4>, N, std::min(256, cdiv(W / 4, 32) * 32), 0, s.x, (AT*)s.hA, a, N, W);
+		else launch_k(s, k_seq_sandwich<AT, 1>, N, std::min(256, cdiv(W, 32) * 32), 0, s.x, (AT*)s.hA, a, N, W);
+	});
+}
 // post-norm blocks: x += norm(y), y = base + the routed experts' sum; the new rows also leave in the activation type (hA), the next sublayer's input
 template <typename AT>
 void post_norm(Seq& s, const float* base, const HcMoe& moe, const SeqNorm& nm, int N) {
@@ -666,8 +715,8 @@ template <typename AT>
 void mixer_typed(Seq& s, const SeqLayer& L, RunState& r, const SeqBatch& sb, double kv_rows, int longest, const OutEpi& oe, const float* proj_in = nullptr, int ld_in = 0) {
 	// proj_in: the mixer's input projection has been computed already (a pair's stacked product): its fp32 columns start there, row stride ld_in,
 	// and a gated-linear-attention's decay input (its last rows) waits in a1 in the activation type
-	const int N = sb.N, W = s.m.width, P = proj_in ? ld_in : proj_stride(L);
-	const float* const proj = proj_in ? proj_in : s.proj;
+	const int N = sb.N, W = s.m.width, gc = gate_cols(s.m), P = proj_in ? ld_in : mixer_stride(s.m, L);
+	const float* const proj = proj_in ? proj_in : s.proj + gc; // behind the residual gate's columns, where the block has one
 	AT *hA = (AT*)s.hA, *a1 = (AT*)s.a1, *a2 = (AT*)s.a2;
 	bool a1_ready = proj_in != nullptr;
 	if (L.type != SEQ_PAIR && !proj_in) {
@@ -675,7 +724,7 @@ void mixer_typed(Seq& s, const SeqLayer& L, RunState& r, const SeqBatch& sb, dou
 		// the mixer's) or the dense unit's up rows (leaving as relu^2 in the activation type)
 		GemmExtra gx;
 		gx.bias = L.b_in;
-		int M = (int)in_rows(L);
+		int M = gc + (int)in_rows(L);
 		if (L.in_tail > 0 && L.ff_kind == SEQ_FF_MOE) M += L.in_tail;
 		if (L.in_tail > 0 && L.ff_kind == SEQ_FF_RELU2) gx.split = M, gx.Y2 = s.ah, gx.ldy2 = L.ff, M += L.in_tail;
 		if (L.in_tail == 0 && L.type == SEQ_GLA) // the decay's low-rank input (the last rows) leaves the epilogue in the activation type, ready for its second product
@@ -683,19 +732,43 @@ void mixer_typed(Seq& s, const SeqLayer& L, RunState& r, const SeqBatch& sb, dou
 		gemm(s, hA, W, 0, L.w_in, W, 0, s.proj, P, 0, N, M, W, 1, EPI_F32, nullptr, -1, true, &gx);
 	}
 	if (L.type == SEQ_LATENT) {
-		const int H = L.heads, D = L.dim, Dv = L.vdim, Rq = L.q_rank, Rk = L.kv_rank;
+		const int H = L.heads, D = L.dim, Dv = L.vdim, Rq = L.q_rank, Rk = L.kv_rank, Pr = L.rot_dims, kd = Rk + Pr;
 		RmsSeg sq{0, Rq, (const bf16*)L.dq_norm}, sc{Rq, Rk, (const bf16*)L.dkv_norm};
-		run_kernel(s, KD_NORM, (double)N * (Rq + Rk) * 8, 0,
-		           [&] { launch_k(s, k_seq_latent_norm<AT>, dim3(cdiv(N, 4), 2), 128, 0, s.proj, P, sq, sc, a1, r.cache_a, sb, s.m.eps); });
-		gemm(s, a1, Rq, 0, L.w_uq, Rq, 0, a2, (long)H * D, 0, N, H * D, Rq, 1, EPI_ACT);
+		const auto rt = s.rot.find(&L);
+		const PairRope rope{Pr, rt == s.rot.end() ? nullptr : rt->second.first, rt == s.rot.end() ? 1.f : rt->second.second};
+		const bool own = !L.kv_shared; // a layer that reads another one's cache has only its query latent to norm
+		run_kernel(s, KD_NORM, (double)N * (Rq + (own ? kd : 0)) * 8, 0,
+		           [&] { launch_k(s, k_seq_latent_norm<AT>, dim3(cdiv(N, 4), own ? 2 : 1), 128, 0, proj, P, sq, sc, a1, r.cache_a, rope, sb, s.m.eps); });
+		if (Pr > 0) { // one product for both parts of the queries: the rotated channels stay fp32, the others leave in the activation type
+			GemmExtra ux;
+			ux.split = H * Pr, ux.split_act = 1, ux.Y2 = a2, ux.ldy2 = (long)H * D;
+			gemm(s, a1, Rq, 0, L.w_uq, Rq, 0, s.f[1], (long)H * Pr, 0, N, H * (Pr + D), Rq, 1, EPI_F32, nullptr, -1, true, &ux);
+			run_kernel(s, KD_QK, (double)N * H * Pr * 8, 0, [&] { launch_k(s, k_seq_rope_heads, N, 128, (Pr / 2) * sizeof(float2), s.f[0], s.f[1], H, (long)H * kd, kd, Rk, rope, sb); });
+		} else gemm(s, a1, Rq, 0, L.w_uq, Rq, 0, a2, (long)H * D, 0, N, H * D, Rq, 1, EPI_ACT);
 		// the key up-projection moves to the query side: q'_h = W_uk,h^T q_h, so scores and values are taken on the cached latent itself
-		gemm(s, a2, (long)H * D, D, L.w_ukT, D, (long)Rk * D, s.f[0], (long)H * Rk, Rk, N, Rk, D, H, EPI_F32);
+		gemm(s, a2, (long)H * D, D, L.w_ukT, D, (long)Rk * D, s.f[0], (long)H * kd, kd, N, Rk, D, H, EPI_F32);
 		AttArgs a;
-		a.q = s.f[0], a.kc = a.vc = r.cache_a, a.kld = a.vld = Rk, a.heads = H, a.group = H, a.tile = attn_tile(H, Rk, Rk), a.kd = a.vd = Rk, a.window = 0;
-		a.scale = L.scale, a.sink = nullptr, a.gate = s.proj + Rq + Rk, a.ldg = P, a.ghs = 1, a.ges = 0, a.keep_first = 0;
-		attention(s, KD_ATTN_LATENT, a, a1, sb, kv_rows, longest);
+		a.q = s.f[0], a.kc = a.vc = r.cache_a, a.kld = a.vld = kd, a.heads = H, a.group = H, a.tile = attn_tile(H, kd, Rk), a.kd = kd, a.vd = Rk, a.window = L.window;
+		a.scale = L.scale, a.sink = (const bf16*)L.sink, a.gate = L.no_gate ? nullptr : proj + Rq + (own ? kd : 0), a.ldg = P, a.ghs = 1, a.ges = 0, a.keep_first = 0;
+		a.split = L.scores_f32;
+		attention(s, KD_ATTN_LATENT, a, a1, sb, L.window > 0 ? std::min(kv_rows, (double)N * L.window) : kv_rows, longest);
 		gemm(s, a1, (long)H * Rk, Rk, L.w_uv, Rk, (long)Dv * Rk, a2, (long)H * Dv, Dv, N, Dv, Rk, H, EPI_ACT);
 		out_product<AT>(s, a2, L.w_o, N, H * Dv, oe, L.b_o);
+	} else if (L.type == SEQ_MINGRU) {
+		const int D = L.dim;
+		int most = 0; // longest portion of the step
+		for (int b = 0; b < sb.B; ++b) most = std::max(most, s.hb_count[b]);
+		MinGruArgs g;
+		g.proj = proj, g.ldp = P, g.width = D, g.state = r.delta;
+		g.chunk = std::max(64, cdiv(most, 64)); // at most 64 maps to fold
+		const int chunks = cdiv(most, g.chunk);
+		g.carries = chunks;
+		if (chunks > 1) ensure_carry(s, (size_t)sb.B * chunks * D);
+		g.carry = s.carry;
+		const dim3 grid(cdiv(D, 64), chunks, sb.B);
+		if (chunks > 1) run_kernel(s, KD_MINGRU, 0, 0, [&] { launch_k(s, k_seq_mingru_chunk, grid, 64, 0, g, sb); });
+		run_kernel(s, KD_MINGRU, (double)N * D * (12 + sizeof(AT)) + 2.0 * sb.B * D * 4, 0, [&] { launch_k(s, k_seq_mingru_apply<AT>, grid, 64, 0, g, a2, sb); });
+		out_product<AT>(s, a2, L.w_o, N, D, oe, L.b_o);
 	} else if (L.type == SEQ_DELTA) {
 		const int H = L.heads, G = L.kv_heads, D = L.dim, Dv = L.vdim;
 		const int cq = 0, ck = G * D, cv = 2 * G * D, cb = cv + H * Dv, ca1 = cb + H, cg1 = ca1 + L.a_rank;
@@ -703,14 +776,14 @@ void mixer_typed(Seq& s, const SeqLayer& L, RunState& r, const SeqBatch& sb, dou
 		ca.seg[0] = ConvSeg{cq, G, D, 1, 1, 1.f / sqrtf((float)D), 0, s.f[0]};
 		ca.seg[1] = ConvSeg{ck, G, D, 1, 1, 1.f, 0, s.f[1]};
 		ca.seg[2] = ConvSeg{cv, H, Dv, 1, 0, 1.f, 0, s.f[2]};
-		conv(s, L, r, ca, sb);
+		conv(s, L, r, ca, sb, proj, P);
 		const int lr = L.a_rank + L.g_rank;
-		run_kernel(s, KD_ELEMENT, (double)N * lr * 6, 0, [&] { launch_k(s, k_seq_cast_cols<AT>, cdiv((long)N * lr, 256), 256, 0, a1, s.proj, P, ca1, lr, N); });
+		run_kernel(s, KD_ELEMENT, (double)N * lr * 6, 0, [&] { launch_k(s, k_seq_cast_cols<AT>, cdiv((long)N * lr, 256), 256, 0, a1, proj, P, ca1, lr, N); });
 		gemm(s, a1, lr, 0, L.w_a2, L.a_rank, 0, s.f[3], (long)H * D, 0, N, H * D, L.a_rank, 1, EPI_F32);
 		gemm(s, a1 + L.a_rank, lr, 0, L.w_g2, L.g_rank, 0, s.f[4], (long)H * Dv, 0, N, H * Dv, L.g_rank, 1, EPI_F32);
 		(void)cg1;
 		DeltaArgs d;
-		d.q = s.f[0], d.k = s.f[1], d.v = s.f[2], d.proj = s.proj, d.ldp = P, d.bcol = cb, d.dt = s.f[3], d.a_log = (const bf16*)L.a_log, d.dt_bias = (const bf16*)L.dt_bias;
+		d.q = s.f[0], d.k = s.f[1], d.v = s.f[2], d.proj = proj, d.ldp = P, d.bcol = cb, d.dt = s.f[3], d.a_log = (const bf16*)L.a_log, d.dt_bias = (const bf16*)L.dt_bias;
 		d.state = r.delta, d.o = s.f[5], d.heads = H, d.kv_heads = G, d.dim = D, d.vdim = Dv;
 		const size_t smem = ((size_t)D * Dv + 3 * D) * sizeof(float);
 		const int threads = std::max(64, cdiv(Dv, 32) * 32);
@@ -769,17 +842,17 @@ void mixer_typed(Seq& s, const SeqLayer& L, RunState& r, const SeqBatch& sb, dou
 		const int H = L.heads, D = L.dim, Dv = L.vdim, Vs = lin_vs(L), ldl = 2 * H * D + H * Vs;
 		LinPack lp;
 		memset(&lp, 0, sizeof(lp));
-		lp.proj = s.proj, lp.ldp = P, lp.lin = s.lin, lp.decay = s.f[3], lp.heads = H, lp.dim = D, lp.vdim = Dv, lp.vs = Vs;
+		lp.proj = proj, lp.ldp = P, lp.lin = s.lin, lp.decay = s.f[3], lp.heads = H, lp.dim = D, lp.vdim = Dv, lp.vs = Vs;
 		LinOut lo;
 		memset(&lo, 0, sizeof(lo));
 		lo.o = s.f[5], lo.ldo = H * Vs, lo.ohs = Vs, lo.heads = H, lo.vdim = Dv, lo.unit = Dv, lo.w = (const bf16*)L.out_norm, lo.eps = s.m.eps, lo.mul = 1.f;
 		float qscale = 1.f;
 		if (L.type == SEQ_MLSTM) {
 			const int cq = 0, ck = H * D, cv = 2 * H * D, cg = cv + H * Dv, ci = cg + H * Dv, cf = ci + H;
-			MlstmGates mg{s.proj, P, ci, cf, H, L.gate_cap, r.mstate, s.f[0], s.f[1], s.f[2]};
+			MlstmGates mg{proj, P, ci, cf, H, L.gate_cap, r.mstate, s.f[0], s.f[1], s.f[2]};
 			run_kernel(s, KD_LINPREP, (double)N * H * 20, 0, [&] { launch_k(s, k_seq_mlstm_gates, dim3(sb.B, H), 32, 0, mg, sb); });
 			lp.mode = LIN_MLSTM, lp.qcol = cq, lp.kcol = ck, lp.vcol = cv, lp.keep = s.f[0], lp.take = s.f[1];
-			lo.w_mod = H * Dv, lo.gate = s.proj + cg, lo.ldg = P, lo.gate_mode = 1, lo.m_t = s.f[2];
+			lo.w_mod = H * Dv, lo.gate = proj + cg, lo.ldg = P, lo.gate_mode = 1, lo.m_t = s.f[2];
 			qscale = 1.f / sqrtf((float)D);
 		} else if (L.type == SEQ_HGRN2) {
 			lp.mode = LIN_HGRN2, lp.qcol = 0, lp.kcol = H * D, lp.vcol = 2 * H * D, lp.lower = (const bf16*)L.lower;
@@ -790,10 +863,10 @@ void mixer_typed(Seq& s, const SeqLayer& L, RunState& r, const SeqBatch& sb, dou
 			ca.seg[0] = ConvSeg{0, H, Dv, 1, 0, 1.f, 0, s.f[0]};
 			ca.seg[1] = ConvSeg{inner, G, D, 1, 0, 1.f, 0, s.f[1]};
 			ca.seg[2] = ConvSeg{inner + G * D, G, D, 1, 0, 1.f, 0, s.f[2]};
-			conv(s, L, r, ca, sb);
+			conv(s, L, r, ca, sb, proj, P);
 			lp.mode = LIN_MAMBA2, lp.xs = s.f[0], lp.bs = s.f[1], lp.cs = s.f[2], lp.dtcol = 2 * inner + 2 * G * D, lp.groups = G;
 			lp.dt_bias = (const bf16*)L.dt_bias, lp.a_log = (const bf16*)L.a_log;
-			lo.unit = inner / L.norm_groups, lo.w_mod = inner, lo.gate = s.proj, lo.ldg = P, lo.gate_mode = 3, lo.skip = s.f[0], lo.skip_w = (const bf16*)L.skip_d;
+			lo.unit = inner / L.norm_groups, lo.w_mod = inner, lo.gate = proj, lo.ldg = P, lo.gate_mode = 3, lo.skip = s.f[0], lo.skip_w = (const bf16*)L.skip_d;
 		}
 		run_kernel(s, KD_LINPREP, (double)N * (ldl + H * D) * 8, 0, [&] { launch_k(s, k_seq_lin_pack, dim3(N, H), 64, 0, lp, N); });
 		GlaArgs g;
@@ -827,7 +900,7 @@ void mixer_typed(Seq& s, const SeqLayer& L, RunState& r, const SeqBatch& sb, dou
 		ca.seg[0] = ConvSeg{0, H, D, 0, 2, 1.f, 0, s.f[0]};
 		ca.seg[1] = ConvSeg{H * D, G, D, 0, 2, 1.f, 1, r.cache_a};
 		ca.seg[2] = ConvSeg{H * D + G * D, G, Dv, 0, 0, 1.f, 1, r.cache_b};
-		conv(s, L, r, ca, sb);
+		conv(s, L, r, ca, sb, proj, P);
 		AttArgs a;
 		a.q = s.f[0], a.kc = r.cache_a, a.vc = r.cache_b, a.kld = G * D, a.vld = G * Dv, a.heads = H, a.group = H / G, a.tile = attn_tile(H / G, D, Dv), a.kd = D, a.vd = Dv;
 		a.window = L.window, a.scale = L.scale, a.sink = (const bf16*)L.sink, a.gate = nullptr, a.ldg = 0, a.ghs = 1, a.ges = 0, a.keep_first = 0;
@@ -881,9 +954,11 @@ void feed_forward(Seq& s, const SeqLayer& L, const SeqBatch& sb, const OutEpi& o
 			gemm(s, hA, W, 0, L.w_sh_gate_up, W, 0, s.fsh, ldsh, 0, N, ldsh, W, 1, EPI_F32);
 			logits = s.fsh + 2 * sf, ldl = ldsh;
 		} else {
+			const int gc = gate_cols(s.m); // sandwich blocks with a residual gate: its rows lead the router's
+			ldl = gc ? gated_stride(s.m, Et) : Et, logits = s.proj + gc;
 			GemmExtra rx;
 			rx.bias = L.b_router;
-			gemm(s, hA, W, 0, L.w_router, W, 0, s.proj, Et, 0, N, Et, W, 1, EPI_F32, nullptr, -1, true, &rx);
+			gemm(s, hA, W, 0, L.w_router, W, 0, s.proj, ldl, 0, N, gc + Et, W, 1, EPI_F32, nullptr, -1, true, &rx);
 		}
 		const float rscale = L.route_scale != 0.f ? L.route_scale : 1.f;
 		// identity experts get groups of their own behind the real ones: their rows are placed but no product runs over them
@@ -934,8 +1009,14 @@ void feed_forward(Seq& s, const SeqLayer& L, const SeqBatch& sb, const OutEpi& o
 			return;
 		}
 		run_kernel(s, KD_ELEMENT, (double)pairs * ff * (8 + sizeof(AT)), 0,
-		           [&] { launch_k(s, k_seq_ff_act<AT>, cdiv((long)pairs * ff, 256), 256, 0, (AT*)s.moe_a, s.moe_y, ff, pairs, 0.f, 1, 2 * ff); });
+		           [&] { launch_k(s, k_seq_ff_act<AT>, cdiv((long)pairs * ff, 256), 256, 0, (AT*)s.moe_a, s.moe_y, ff, pairs, L.limit, L.expert_act == 2 ? 0 : 1, 2 * ff); });
 		gemm(s, s.moe_a, ff, 0, L.w_down, ff, (long)W * ff, s.moe_d, W, 0, N, W, ff, E, EPI_F32, nullptr, -1, true, &gx);
+		if (oe.sand) { // sandwich blocks: the weighted sum is formed by the kernel that gates and norms it
+			Sandwich a = *oe.sand;
+			a.base = nullptr, a.moe = HcMoe{s.moe_d, s.moe_inv, s.moe_sel, s.moe_wt, top, E};
+			sandwich<AT>(s, a, N);
+			return;
+		}
 		if (oe.post) { // post-norm blocks: the weighted sum is formed by the kernel that norms it and adds it to the stream
 			post_norm<AT>(s, nullptr, HcMoe{s.moe_d, s.moe_inv, s.moe_sel, s.moe_wt, top, E}, *oe.post, N);
 			return;
@@ -986,6 +1067,42 @@ void layer_typed(Seq& s, const SeqLayer& L, RunState& r, const SeqBatch& sb, dou
 		}
 		return;
 	}
+	if (s.m.block == SEQ_BLOCK_SANDWICH) {
+		// every sublayer's input is written by the kernel that ends the one before it; only the step's first is a norm of its own
+		if (!s.h_ready) norm(s, s.hA, s.x, nullptr, L.norm1, N);
+		Sandwich a;
+		memset(&a, 0, sizeof(a));
+		a.offset = s.m.norm_offset, a.eps = s.m.eps, a.hist = s.hist, a.k = r.layer + 1;
+		auto ends_layer = [&] { a.dwa = (const bf16*)L.dwa, a.w_next = next ? (const bf16*)next->norm1.w : nullptr; };
+		mixer_typed<AT>(s, L, r, sb, kv_rows, longest, OutEpi{EPI_F32, nullptr, s.mo, nullptr});
+		a.base = s.mo, a.w = (const bf16*)L.norm1b.w;
+		if (gate_cols(s.m)) a.gate = s.proj, a.ldg = mixer_stride(s.m, L);
+		if (L.ff > 0) a.w_next = (const bf16*)L.norm2.w;
+		else ends_layer();
+		sandwich<AT>(s, a, N);
+		if (L.ff > 0) {
+			OutEpi oe{EPI_F32, nullptr, s.mo, nullptr};
+			a.w = (const bf16*)L.norm2b.w;
+			ends_layer();
+			if (L.ff_kind == SEQ_FF_MOE) {
+				if (gate_cols(s.m)) a.gate = s.proj, a.ldg = gated_stride(s.m, L.experts + L.ident);
+				oe.sand = &a;
+				feed_forward<AT>(s, L, sb, oe);
+			} else {
+				if (gate_cols(s.m)) {
+					const int W = s.m.width;
+					GemmExtra gx;
+					gx.bias = L.b_rg2;
+					gemm(s, s.hA, W, 0, L.w_rg2, W, 0, s.fsh, W, 0, N, W, W, 1, EPI_F32, nullptr, -1, true, &gx);
+					a.gate = s.fsh, a.ldg = W;
+				}
+				feed_forward<AT>(s, L, sb, oe);
+				sandwich<AT>(s, a, N);
+			}
+		}
+		s.h_ready = next != nullptr;
+		return;
+	}
 	norm(s, s.hA, s.x, nullptr, L.norm1, N);
 	if (s.m.block == SEQ_BLOCK_SERIAL) {
 		mixer_typed<AT>(s, L, r, sb, kv_rows, longest, OutEpi{EPI_DYT_RES, &L.norm1b, s.x, nullptr});
@@ -1007,8 +1124,8 @@ void forward(Seq& s, const SeqBatch& sb, int n_want, double kv_rows, int longest
 	const int N = sb.N;
 	const bool looped = m.loop_times > 1;
 	s.h_ready = false;
-	run_kernel(s, KD_EMBED, (double)N * m.width * (2.0 + (m.pos_table ? 2.0 : 0.0) + (m.bigram ? 2.0 : 0.0) + 4.0 * s.streams + (looped ? 4.0 : 0.0)), 0,
-	           [&] { launch_k(s, k_seq_embed, N, 128, 0, s.x, looped ? s.x0 : nullptr, (const bf16*)m.embed, s.d_tok, N, m.width, m.embed_scale != 0.f ? m.embed_scale : 1.f, (const bf16*)m.pos_table, s.d_tpos, s.streams,
+	run_kernel(s, KD_EMBED, (double)N * m.width * (2.0 + (m.pos_table ? 2.0 : 0.0) + (m.bigram ? 2.0 : 0.0) + 4.0 * s.streams + (looped || s.depth ? 4.0 : 0.0)), 0,
+	           [&] { launch_k(s, k_seq_embed, N, 128, 0, s.x, looped ? s.x0 : s.depth ? s.hist : nullptr, (const bf16*)m.embed, s.d_tok, N, m.width, m.embed_scale != 0.f ? m.embed_scale : 1.f, (const bf16*)m.pos_table, s.d_tpos, s.streams,
 	                          EmbedBigram{(const bf16*)m.bigram, s.d_tprev, m.bigram_buckets, m.bigram_mul_prev, m.bigram_mul_cur}); });
 	for (size_t ri = 0; ri < s.runs.size(); ++ri) {
 		RunState& r = s.runs[ri];
@@ -1043,7 +1160,7 @@ void forward_decode_graph(Seq& s, const SeqBatch& sb, int n_want, double kv_rows
 	auto one = [&](const SeqLayer& L) {
 		if (L.type != SEQ_LATENT && L.type != SEQ_WINDOW && L.type != SEQ_GQA) return; // recurrent mixers: nothing to share out
 		const bool lat = L.type == SEQ_LATENT;
-		const int group = lat ? L.heads : L.heads / L.kv_heads, kd = lat ? L.kv_rank : L.dim, vd = lat ? L.kv_rank : L.vdim;
+		const int group = lat ? L.heads : L.heads / L.kv_heads, kd = lat ? L.kv_rank + L.rot_dims : L.dim, vd = lat ? L.kv_rank : L.vdim;
 		const int ns = attn_nsplit(s, sb.N, L.heads / attn_tile(group, kd, vd), attn_span(L), longest);
 		key.push_back(ns);
 		part_need = std::max(part_need, (size_t)sb.N * L.heads * ns * (vd + 2));
@@ -1143,7 +1260,16 @@ extern "C" void* calm_b200_seq_prepare(const struct SeqModel* model) {
 			give(r.sub[0], L.pair[0]), give(r.sub[1], L.pair[1]);
 			return;
 		}
-		if (L.type == SEQ_LATENT) r.cache_a = (float*)dalloc(rows * L.kv_rank * sizeof(float));
+		if (L.type == SEQ_LATENT) {
+			if (L.kv_shared) { // the rows an earlier layer caches (outside loops a layer is one run)
+				for (const RunState& o : s.runs)
+					if (o.layer == L.kv_shared - 1) r.cache_a = o.cache_a, r.cache_borrowed = true;
+			} else r.cache_a = (float*)dalloc(rows * (L.kv_rank + L.rot_dims) * sizeof(float));
+		}
+		if (L.type == SEQ_MINGRU) {
+			r.delta_per_slot = L.dim;
+			r.delta = (float*)dalloc(r.delta_per_slot * m.max_seqs * sizeof(float));
+		}
 		if (L.type == SEQ_WINDOW || L.type == SEQ_GQA) {
 			r.cache_a = (float*)dalloc(rows * L.kv_heads * L.dim * sizeof(float));
 			r.cache_b = (float*)dalloc(rows * L.kv_heads * L.vdim * sizeof(float));
@@ -1180,13 +1306,13 @@ extern "C" void* calm_b200_seq_prepare(const struct SeqModel* model) {
 	});
 	CUDA_CHECK(cudaFuncSetAttribute(k_seq_attention<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024));
 	CUDA_CHECK(cudaFuncSetAttribute(k_seq_attention<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024));
-	// rotation tables of the grouped-query attentions: angle step per rotated pair (in double), rescaled between two wavelengths
+	// rotation tables of the grouped-query and latent attentions: angle step per rotated pair (in double), rescaled between two wavelengths
 	std::function<void(const SeqLayer&)> rot_table = [&](const SeqLayer& L) {
 		if (L.type == SEQ_PAIR) {
 			rot_table(L.pair[0]), rot_table(L.pair[1]);
 			return;
 		}
-		if (L.type != SEQ_GQA || L.rot_dims < 2) return;
+		if ((L.type != SEQ_GQA && L.type != SEQ_LATENT) || L.rot_dims < 2) return;
 		const int dims = L.rot_dims, half = dims / 2;
 		std::vector<double> f(half);
 		float mag = 1.f;
@@ -1207,6 +1333,7 @@ extern "C" void* calm_b200_seq_prepare(const struct SeqModel* model) {
 		s.rot[&L] = std::make_pair(dev, mag);
 	};
 	for (const SeqLayer& L : s.layers) rot_table(L);
+	for (const SeqLayer& L : s.layers) s.depth |= L.dwa != nullptr;
 	// workspace widths
 	std::function<void(const SeqLayer&)> widths = [&](const SeqLayer& L) {
 		if (L.type == SEQ_PAIR) {
@@ -1216,7 +1343,7 @@ extern "C" void* calm_b200_seq_prepare(const struct SeqModel* model) {
 		}
 		if (L.ff > 0 && L.ff_kind == SEQ_FF_MOE) {
 			s.max_top = std::max(s.max_top, L.top), s.max_experts = std::max(s.max_experts, L.experts + L.ident), s.w_moe_ff = std::max(s.w_moe_ff, (size_t)L.ff);
-			s.w_proj = std::max(s.w_proj, (size_t)L.experts + L.ident);
+			s.w_proj = std::max(s.w_proj, (size_t)gated_stride(m, L.experts + L.ident));
 			if (L.shared_ff > 0) s.w_fsh = std::max(s.w_fsh, (size_t)2 * L.shared_ff + 1 + L.experts + L.ident);
 			s.w_a = std::max(s.w_a, (size_t)L.shared_ff);
 		}
@@ -1227,11 +1354,13 @@ extern "C" void* calm_b200_seq_prepare(const struct SeqModel* model) {
 			s.w_a = std::max(s.w_a, (size_t)L.heads * L.vdim);
 			s.w_lin = std::max(s.w_lin, (size_t)2 * L.heads * L.dim + (size_t)L.heads * lin_vs(L));
 		}
-		s.w_proj = std::max({s.w_proj, (size_t)proj_stride(L), (size_t)2 * L.ff});
+		s.w_proj = std::max({s.w_proj, (size_t)mixer_stride(m, L), (size_t)2 * L.ff});
+		if (L.w_rg2) s.w_fsh = std::max(s.w_fsh, (size_t)m.width);
 		if (L.ff > 0 && L.ff_kind == SEQ_FF_RELU2 && L.in_tail > 0) s.w_ah = std::max(s.w_ah, (size_t)L.ff);
 		size_t wf = 0, wa = (size_t)L.ff;
-		if (L.type == SEQ_LATENT) wf = (size_t)L.heads * L.kv_rank, wa = std::max({wa, (size_t)L.heads * L.kv_rank, (size_t)L.heads * L.dim, (size_t)L.heads * L.vdim, (size_t)L.q_rank});
+		if (L.type == SEQ_LATENT) wf = (size_t)L.heads * (L.kv_rank + L.rot_dims), wa = std::max({wa, (size_t)L.heads * (L.kv_rank + L.rot_dims) * (L.scores_f32 ? 3 : 1), (size_t)L.heads * L.dim, (size_t)L.heads * L.vdim, (size_t)L.q_rank});
 		if (L.type == SEQ_DELTA) wf = std::max((size_t)L.heads * L.dim, (size_t)L.heads * L.vdim), wa = std::max({wa, (size_t)L.heads * L.vdim, (size_t)L.a_rank + L.g_rank});
+		if (L.type == SEQ_MINGRU) wa = std::max(wa, (size_t)L.dim);
 		if (L.type == SEQ_WINDOW) wf = (size_t)L.heads * L.dim, wa = std::max({wa, (size_t)L.heads * L.vdim, (size_t)L.heads * L.dim});
 		s.w_f = std::max(s.w_f, wf), s.w_a = std::max(s.w_a, wa);
 	};
@@ -1252,11 +1381,12 @@ extern "C" void calm_b200_seq_release(void* handle) {
 	cudaStreamSynchronize(s->stream);
 	drop_graphs(*s);
 	std::function<void(RunState&)> drop = [&](RunState& r) {
-		cudaFree(r.cache_a), cudaFree(r.cache_b), cudaFree(r.conv), cudaFree(r.delta), cudaFree(r.mstate), cudaFree(r.slopes);
+		if (!r.cache_borrowed) cudaFree(r.cache_a);
+		cudaFree(r.cache_b), cudaFree(r.conv), cudaFree(r.delta), cudaFree(r.mstate), cudaFree(r.slopes);
 		for (RunState& q : r.sub) drop(q);
 	};
 	for (RunState& r : s->runs) drop(r);
-	cudaFree(s->lin), cudaFree(s->fsh);
+	cudaFree(s->lin), cudaFree(s->fsh), cudaFree(s->hist), cudaFree(s->carry);
 	cudaFree(s->table_dev), cudaFree(s->d_tok), cudaFree(s->d_want), cudaFree(s->d_argmax), cudaFree(s->logits), cudaFree(s->hW);
 	cudaFree(s->part), cudaFree(s->a3), cudaFree(s->att_kb), cudaFree(s->att_vt), cudaFree(s->att_s), cudaFree(s->att_p), cudaFree(s->x), cudaFree(s->x0), cudaFree(s->proj), cudaFree(s->hA), cudaFree(s->a1), cudaFree(s->a2), cudaFree(s->trace_buf);
 	for (float* p : s->f) cudaFree(p);

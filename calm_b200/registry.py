@@ -17,12 +17,13 @@ def register(architecture: str, loader: Callable) -> None:
 
 
 def _defaults() -> None:
-    from . import bovinex, sopepel, vimulorn, zazilix
+    from . import bovinex, fasulix, sopepel, vimulorn, zazilix
 
     register(vimulorn.ARCHITECTURE, vimulorn.load)
     register(bovinex.ARCHITECTURE, bovinex.load)
     register(zazilix.ARCHITECTURE, zazilix.load)
     register(sopepel.ARCHITECTURE, sopepel.load)
+    register(fasulix.ARCHITECTURE, fasulix.load)
 
 
 def architecture_of(path: str) -> str:

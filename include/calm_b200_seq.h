@@ -60,6 +60,17 @@
  * route_mode 2 -- scores are sigmoid(router output), the `top` highest are taken, the weights are those scores times route_scale,
  * not renormalised; `weight_input` -- the weight multiplies the expert's input instead of its output; `shared_gate` -- the shared
  * unit's output is multiplied by sigmoid(one more row of its first product), one number per token.
+ * Sandwich blocks (SEQ_BLOCK_SANDWICH): the model's RMS norm before and after every sublayer, x <- x + norm1b(mixer(norm1(x))), then
+ * x <- x + norm2b(feed-forward(norm2(x))).  With SeqModel.res_gate a sublayer's output is multiplied, before its second norm, by
+ * sigmoid(R h + r) column by column, h being the sublayer's normed input: R's `width` rows (and r) lead w_in / b_in, and for routed
+ * experts w_router / b_router (other feed-forwards: w_rg2 / b_rg2).  SeqLayer.dwa averages over depth: with X_0 the embedding rows and
+ * X_(k+1) the stream as layer k leaves it, what goes on after layer i is sum_(j <= i+1) dwa[j] X_j.
+ * Mixer SEQ_MINGRU: dim channels (heads 1, vdim = dim), each S <- (1 - z) S + z c with z = sigmoid(.) and c = u + 1/2 (u >= 0) or
+ * sigmoid(u) (u < 0) read from the current token alone, z and u biased (b_in); output S silu(g).
+ * Options of SEQ_LATENT: rot_dims > 0 -- every head has rot_dims more query channels, and one more key part of rot_dims channels, shared by
+ * the heads, is cached behind the latent; both turn by the position, channels 2i and 2i + 1 together; `window`, `sink` and `scores_f32` as
+ * for the other attentions; `no_gate` -- no gate rows; `kv_shared` -- the layer has no key/value latent of its own and reads the cache of an earlier one.
+ * expert_act 2 -- a routed expert is the clamped gated unit (SeqLayer.limit).
  * Embedding: SeqModel.bigram adds row (previous token * mul_prev + token * mul_cur) mod buckets of a second table (row `buckets`
  * for a sequence's first token); the previous token is kept with the sequence's slot.  SeqModel.logit_scale multiplies the logits.
  */
@@ -73,9 +84,9 @@
 extern "C" {
 #endif
 
-enum SeqMixer { SEQ_LATENT = 0, SEQ_DELTA = 1, SEQ_WINDOW = 2, SEQ_GQA = 3, SEQ_GLA = 4, SEQ_MLSTM = 5, SEQ_HGRN2 = 6, SEQ_MAMBA2 = 7, SEQ_PAIR = 8 };
+enum SeqMixer { SEQ_LATENT = 0, SEQ_DELTA = 1, SEQ_WINDOW = 2, SEQ_GQA = 3, SEQ_GLA = 4, SEQ_MLSTM = 5, SEQ_HGRN2 = 6, SEQ_MAMBA2 = 7, SEQ_PAIR = 8, SEQ_MINGRU = 9 };
 enum SeqNormKind { SEQ_NORM_DYT = 0, SEQ_NORM_RMS = 1 };
-enum SeqBlock { SEQ_BLOCK_SERIAL = 0, SEQ_BLOCK_PARALLEL = 1, SEQ_BLOCK_HYPER = 2, SEQ_BLOCK_POST = 3 };
+enum SeqBlock { SEQ_BLOCK_SERIAL = 0, SEQ_BLOCK_PARALLEL = 1, SEQ_BLOCK_HYPER = 2, SEQ_BLOCK_POST = 3, SEQ_BLOCK_SANDWICH = 4 };
 enum SeqFfKind { SEQ_FF_CLAMPED = 0, SEQ_FF_RELU2 = 1, SEQ_FF_MOE = 2, SEQ_FF_GATED = 3 };
 enum SeqFfAct { SEQ_ACT_SILU = 0, SEQ_ACT_GELU_TANH = 1 };
 
@@ -101,13 +112,13 @@ struct SeqLayer {
 	int dim, vdim;       /* per-head query/key width and value width */
 	int q_rank, kv_rank; /* SEQ_LATENT */
 	int taps;            /* SEQ_DELTA / SEQ_WINDOW: convolution taps (1 = none) */
-	int window;          /* SEQ_WINDOW: positions seen, the current one included; <= 0: unbounded */
+	int window;          /* SEQ_WINDOW / SEQ_GQA / SEQ_LATENT: positions seen, the current one included; <= 0: unbounded */
 	int a_rank, g_rank;  /* SEQ_DELTA: inner widths of the decay and gate projections */
 	int ff;              /* feed-forward width, 0 = no feed-forward */
 	float scale;         /* score scale of the attentions */
 	float limit;         /* clamp of the feed-forward */
 	struct SeqNorm norm1, norm1b, norm2, norm2b;
-	/* SEQ_LATENT: rows [dq | dkv | g];  SEQ_DELTA: [q | k | v | b | a1 | g1];  SEQ_WINDOW: [q | k | v];
+	/* SEQ_LATENT: rows [dq | dkv | rotated key part | g] (kv_shared: [dq | g]; no_gate: without g);  SEQ_MINGRU: [z | x | g];  SEQ_DELTA: [q | k | v | b | a1 | g1];  SEQ_WINDOW: [q | k | v];
 	 * SEQ_GQA: [q | k | v | g] (no_gate: [q | k | v]);  SEQ_GLA: [q | k | v | g | a1];  SEQ_MLSTM: [q | k | v | g | i | f];
 	 * SEQ_HGRN2: [q | f | v];  SEQ_MAMBA2: [z | x | B | C | dt] */
 	const void* w_in;
@@ -115,7 +126,7 @@ struct SeqLayer {
 	/* SEQ_LATENT */
 	const void* dq_norm;   /* bf16 [q_rank] */
 	const void* dkv_norm;  /* bf16 [kv_rank] */
-	const void* w_uq;      /* (heads*dim, q_rank) */
+	const void* w_uq;      /* (heads*dim, q_rank); with rot_dims: (heads*(rot_dims + dim), q_rank), the rotated rows of all heads, then the unrotated rows of all heads */
 	const void* w_ukT;     /* per head the TRANSPOSED key up-projection: [heads][kv_rank][dim] */
 	const void* w_uv;      /* (heads*vdim, kv_rank) */
 	/* SEQ_DELTA / SEQ_WINDOW */
@@ -127,7 +138,7 @@ struct SeqLayer {
 	const void* dt_bias;   /* bf16 [heads*dim] */
 	const void* out_norm;  /* bf16 [vdim] */
 	/* SEQ_WINDOW */
-	const void* sink;      /* bf16 [heads] or NULL */
+	const void* sink;      /* bf16 [heads] or NULL (also SEQ_LATENT) */
 	/* feed-forward */
 	const void* w_gate_up; /* rows [gate | up]: (2*ff, width); SEQ_FF_RELU2: up only (ff, width); SEQ_FF_MOE: [experts](2*ff, width) */
 	const void* w_down;    /* (width, ff); SEQ_FF_MOE: [experts](width, ff) */
@@ -137,7 +148,7 @@ struct SeqLayer {
 	const void* k_norm;    /* SEQ_GQA: bf16 [kv_heads*dim] */
 	const void* b_a2;      /* SEQ_GLA: bf16 [heads*dim], bias of the decay projection */
 	int keep_first;        /* SEQ_GQA: the first positions every query keeps seeing (with `window`) */
-	int rot_dims;          /* SEQ_GQA: rotated channels per head (even, <= dim; 0: none) */
+	int rot_dims;          /* SEQ_LATENT: rotated channels beside the `dim` unrotated ones (even); SEQ_GQA: rotated channels per head (even, <= dim; 0: none) */
 	float rot_base;
 	float rot_factor;      /* frequency rescaling between two wavelengths; <= 0: none */
 	float rot_original, rot_fast, rot_slow;
@@ -187,9 +198,16 @@ struct SeqLayer {
 	/* SEQ_FF_GATED */
 	int ff_act;            /* enum SeqFfAct: activation of the gate rows (w_gate_up rows [gate | up]) */
 	/* SEQ_FF_MOE, further options */
-	int expert_act;        /* 0: an expert is down(silu(gate) * up), rows [gate | up]; 1: down(relu(up)^2), w_gate_up = [experts](ff, width), the shared unit alike */
+	int expert_act;        /* 0: an expert is down(silu(gate) * up), rows [gate | up]; 1: down(relu(up)^2), w_gate_up = [experts](ff, width), the shared unit alike;
+	                          2: the clamped gated unit, rows [gate | up], clamp `limit` */
 	int weight_input;      /* 1: a choice's weight multiplies the expert's input */
 	int shared_gate;       /* 1: w_sh_gate_up has one more row behind the unit's first rows (before the router's): the shared output is multiplied by its sigmoid */
+	/* SEQ_LATENT, further option */
+	int kv_shared;         /* 0: own key/value latent; k > 0: layer k - 1's cache rows are read (same kv_rank, rot_dims and rotation; that layer has its own) */
+	/* SEQ_BLOCK_SANDWICH */
+	const void* dwa;       /* bf16 [layer index + 2]: weights of the depth average, or NULL: the stream goes on as it is */
+	const void* w_rg2;     /* res_gate, feed-forward other than SEQ_FF_MOE: (width, width) and bf16 [width] or NULL */
+	const void* b_rg2;
 };
 
 struct SeqModel {
@@ -215,6 +233,7 @@ struct SeqModel {
 	const void* bigram; /* bf16 (bigram_buckets + 1, width): rows added to the embedding, picked by a hash of (previous token, token); or NULL */
 	int bigram_buckets, bigram_mul_prev, bigram_mul_cur;
 	float logit_scale;  /* factor on the logits (0 is read as 1) */
+	int res_gate;       /* SEQ_BLOCK_SANDWICH: 1: a sigmoid gate per column on every sublayer's output */
 };
 
 /* cudaMalloc + copy, like upload_cuda */

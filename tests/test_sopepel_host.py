@@ -91,12 +91,12 @@ def test_records_match_the_header():
     body = text[text.index("struct SeqLayer {"):text.index("struct SeqModel {")]
     names = [n for n, _ in seqlib.SeqLayer._fields_]
     tail = ["qk_per_head", "gate_per_head", "b_o", "scores_f32", "ff_act", "expert_act", "weight_input", "shared_gate"]
-    assert names[-len(tail):] == tail
+    assert names[names.index(tail[0]):][:len(tail)] == tail
     at = [body.index(" " + n + ";") for n in tail]
     assert at == sorted(at)
     model = text[text.index("struct SeqModel {"):]
     mnames = [n for n, _ in seqlib.SeqModel._fields_]
-    assert mnames[-5:] == ["bigram", "bigram_buckets", "bigram_mul_prev", "bigram_mul_cur", "logit_scale"]
+    assert mnames[mnames.index("bigram"):][:5] == ["bigram", "bigram_buckets", "bigram_mul_prev", "bigram_mul_cur", "logit_scale"]
     assert model.index("bigram;") < model.index("bigram_buckets, bigram_mul_prev, bigram_mul_cur;") < model.index("logit_scale;")
 
 
