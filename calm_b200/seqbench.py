@@ -3,7 +3,8 @@ model on the same GPU: Vimulorn beside a Llama-shaped stack of the same width, d
 fp16 on the calm engine; Bovinex beside Vimulorn at the same width, depth, head geometry, window and feed-forward width on
 the same runtime (both have windowed grouped-query attention and a recurrent mixer with a [dim x vdim] state per head); Zazilix
 beside Bovinex likewise (both have grouped-query attention with a bounded view, linear recurrences on the same scan kernel and routed experts);
-Sopepel beside Bovinex too (the same two mixers, grouped-query attention and gated linear attention, side by side in every layer with half the heads each).
+Sopepel beside Bovinex too (the same two mixers, grouped-query attention and gated linear attention, side by side in every layer with half the heads each);
+Fasulix beside Vimulorn (latent attention, the clamped unit, a norm before and after every sublayer) and Bovinex (routed experts).
 
 Per size: prompt throughput (one prompt of `prompt` tokens as one step), decode throughput for one sequence and for a
 batch, each after warm-up, timed with CUDA events on the library's stream; then one profiled pass that brackets every
@@ -87,6 +88,21 @@ def sopepel_config(z: dict) -> dict:
             "vocab": z["vocab"], "width": z["width"], "logit_scale": 1.0}
 
 
+def fasulix_config(z: dict) -> dict:
+    """Blocks of [latent attention with a sink, minGRU, latent attention under a window], every layer with eight routed clamped units of half
+    the dense width (two active per token); the windowed layers of later blocks read the first one's latents.  A head is as wide as
+    Vimulorn's, a quarter of it rotated; the recurrence has as many channels as the attention's heads together."""
+    H, D = z["heads"], z["dim"]
+    moe = {"kind": "moe", "expert": {"ff": z["ff"] // 2, "limit": 7.0}, "router": {"experts": 8, "top": 2}}
+    lat = {"heads": H, "dim": D - D // 4, "rot_dim": D // 4, "vdim": D, "kv_rank": z["kv_rank"], "q_rank": z["q_rank"], "scale": D ** -0.5, "rot": {"dims": D // 4, "base": 1e6}}
+    layers = []
+    for b in range(z["blocks"]):
+        win = dict(lat, mask={"size": z["window"]})
+        layers += [{"type": "latent_attention", "mixer": lat, "mlp": moe}, {"type": "mingru", "mixer": {"width": H * D}, "mlp": moe},
+                   {"type": "latent_attention_2", "mixer": win if b == 0 else dict(win, kv_from=2), "mlp": moe}]
+    return {"architecture": "Fasulix", "layers": layers, "norm": {"eps": 1e-5}, "vocab": z["vocab"], "width": z["width"]}
+
+
 def peaks():
     p = os.path.join(ROOT, "MEASURED_PEAKS.json")
     if os.path.exists(p):
@@ -107,11 +123,11 @@ def roofline_table(stats: dict, hbm_gbs: float, tflops: float) -> dict:
 
 
 def bench_family(family: str, name: str, prompt: int, batch: int, steps: int, warmup: int, seed: int = 0) -> list:
-    from . import bovinex, sopepel, vimulorn, zazilix
+    from . import bovinex, fasulix, sopepel, vimulorn, zazilix
 
     z = SIZES[name]
     mod, cfg = {"bovinex": (bovinex, bovinex_config(z)), "zazilix": (zazilix, zazilix_config(z, prompt + steps + 2 * warmup + 64)),
-                "sopepel": (sopepel, sopepel_config(z))}.get(family, (vimulorn, vimulorn_config(z)))
+                "sopepel": (sopepel, sopepel_config(z)), "fasulix": (fasulix, fasulix_config(z))}.get(family, (vimulorn, vimulorn_config(z)))
     hbm, tf, src = peaks()
     t0 = time.time()
     tensors = mod.random_tensors(cfg, seed)
@@ -204,9 +220,9 @@ def main(sizes, prompt=2048, batch=16, steps=32, warmup=8, twin=True, family="vi
     out = []
     for name in sizes:
         lines = bench_family(family, name, prompt, batch, steps, warmup)
-        if twin and family == "bovinex":
+        if twin and family in ("bovinex", "fasulix"):
             lines += bench_family("vimulorn", name, prompt, batch, steps, warmup)
-        if twin and family in ("zazilix", "sopepel"):
+        if twin and family in ("zazilix", "sopepel", "fasulix"):
             lines += bench_family("bovinex", name, prompt, batch, steps, warmup)
         if llama:
             lines += bench_llama_twin(name, prompt, steps, warmup)
