@@ -173,8 +173,9 @@ __global__ void k_seq_latent_norm(const float* proj, int ldp, RmsSeg sq, RmsSeg 
 		}
 	}
 }
-// the rotated query channels of every head: q[n][h * ldh + col + d] from src [N][heads * dims]; one CTA per token, the angles are formed once
-__global__ void __launch_bounds__(128) k_seq_rope_heads(float* q, const float* src, int heads, long ldq, int ldh, int col, PairRope rope, SeqBatch sb) {
+// the rotated query channels of every head: q[n][h * ldh + col + d] from src [N][heads * dims]; one CTA per token, the angles are formed once.
+// qb given: the queries leave in the activation type instead (split3 = 0), or as [hi | hi | lo] rows of split3 columns each (see k_seq_split_q).
+__global__ void __launch_bounds__(128) k_seq_rope_heads(float* q, bf16* qb, int split3, const float* src, int heads, long ldq, int ldh, int col, PairRope rope, SeqBatch sb) {
 	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
 	extern __shared__ float2 cs2[]; // [dims / 2] (cos, sin)
 	const int n = blockIdx.x, half = rope.dims / 2;
@@ -187,8 +188,18 @@ __global__ void __launch_bounds__(128) k_seq_rope_heads(float* q, const float* s
 	for (int e = threadIdx.x; e < heads * half; e += blockDim.x) {
 		const int h = e / half, i = e % half;
 		const float u = src[(size_t)n * heads * rope.dims + 2 * e], v = src[(size_t)n * heads * rope.dims + 2 * e + 1];
-		float* d = q + (size_t)n * ldq + (size_t)h * ldh + col + 2 * i;
-		d[0] = u * cs2[i].x - v * cs2[i].y, d[1] = v * cs2[i].x + u * cs2[i].y;
+		const float r0 = u * cs2[i].x - v * cs2[i].y, r1 = v * cs2[i].x + u * cs2[i].y;
+		if (!qb) {
+			float* d = q + (size_t)n * ldq + (size_t)h * ldh + col + 2 * i;
+			d[0] = r0, d[1] = r1;
+			continue;
+		}
+		bf16* d = qb + (size_t)n * ldq + (size_t)h * ldh + col + 2 * i;
+		d[0] = __float2bfloat16_rn(r0), d[1] = __float2bfloat16_rn(r1);
+		if (split3 > 0) {
+			d[split3] = d[0], d[split3 + 1] = d[1];
+			d[2 * split3] = __float2bfloat16_rn(r0 - __bfloat162float(d[0])), d[2 * split3 + 1] = __float2bfloat16_rn(r1 - __bfloat162float(d[1]));
+		}
 	}
 }
 
@@ -217,25 +228,19 @@ __global__ void k_seq_split_q(bf16* out, const float* q, int kd, size_t units) {
 // feed-forward unit on the stacked [gate | up] product.  mode 0: g = min(gate, L), u = clamp(up, -L, L), y = g sigmoid(1.702 g) (u + 1);
 // mode 1: y = silu(gate) up; mode 2: y = gelu(gate) up, gelu(z) = z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))
 // (ld: row stride of gu, 2 * ff when the product holds nothing else)
+__device__ __forceinline__ float glu_unit(float g, float u, float limit, int mode) {
+	if (mode == 1) return g * sigmoidf_(g) * u;
+	if (mode == 2) return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+	g = fminf(g, limit), u = fminf(fmaxf(u, -limit), limit);
+	return g * sigmoidf_(1.702f * g) * (u + 1.f);
+}
 template <typename AT>
 __global__ void k_seq_ff_act(AT* out, const float* gu, int ff, int N, float limit, int mode, int ld) {
 	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
 	const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
 	if (i >= (size_t)N * ff) return;
 	const size_t n = i / ff, c = i % ff;
-	if (mode == 1) {
-		const float g = gu[n * ld + c];
-		out[i] = to_act<AT>(g * sigmoidf_(g) * gu[n * ld + ff + c]);
-		return;
-	}
-	if (mode == 2) {
-		const float g = gu[n * ld + c];
-		out[i] = to_act<AT>(0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * gu[n * ld + ff + c]);
-		return;
-	}
-	const float g = fminf(gu[n * ld + c], limit);
-	const float u = fminf(fmaxf(gu[n * ld + ff + c], -limit), limit);
-	out[i] = to_act<AT>(g * sigmoidf_(1.702f * g) * (u + 1.f));
+	out[i] = to_act<AT>(glu_unit(gu[n * ld + c], gu[n * ld + ff + c], limit, mode));
 }
 
 // y = silu(gate) up on TWO stacked products in one launch (the routed experts' rows and the shared unit's rows of one feed-forward)
@@ -518,28 +523,211 @@ __global__ void __launch_bounds__(ATT_THREADS) k_seq_attention(AttArgs a, AT* ou
 		}
 	}
 }
-// folds the shares of one (token, head) in share order: one CTA per (token, head)
+// folds the shares of one (token, head) in share order: one CTA per (token, head, 128 value columns)
+#define ATT_MAXSPLIT 128
 template <typename AT>
-__global__ void k_seq_attention_merge(AttArgs a, AT* out) {
+__global__ void __launch_bounds__(128) k_seq_attention_merge(AttArgs a, AT* out) {
 	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
-	const int n = blockIdx.x, h = blockIdx.y, pw = a.vd + 2;
+	__shared__ float wz[ATT_MAXSPLIT], red[2][4];
+	const int n = blockIdx.x, h = blockIdx.y, pw = a.vd + 2, z = threadIdx.x, d = blockIdx.z * 128 + threadIdx.x;
 	if (a.skip && a.skip[n]) return;
 	const float* p = a.part + ((size_t)n * a.heads + h) * a.nsplit * pw;
-	float mx = -INFINITY;
-	for (int z = 0; z < a.nsplit; ++z) mx = fmaxf(mx, p[z * pw + a.vd]);
-	float l = 0.f;
-	for (int z = 0; z < a.nsplit; ++z) {
-		const float m = p[z * pw + a.vd];
-		if (m != -INFINITY) l += p[z * pw + a.vd + 1] * expf(m - mx);
-	}
-	for (int d = threadIdx.x; d < a.vd; d += blockDim.x) {
-		const float g = (a.gate ? sigmoidf_(a.gate[(size_t)n * a.ldg + (size_t)h * a.ghs + (size_t)d * a.ges]) : 1.f) / l;
-		float v = 0.f;
-		for (int z = 0; z < a.nsplit; ++z) {
-			const float m = p[z * pw + a.vd];
-			if (m != -INFINITY) v += p[z * pw + d] * expf(m - mx);
+	const float m = z < a.nsplit ? p[z * pw + a.vd] : -INFINITY, lz = z < a.nsplit ? p[z * pw + a.vd + 1] : 0.f;
+	float mx = warp_max(m);
+	if ((z & 31) == 0) red[0][z >> 5] = mx;
+	__syncthreads();
+	mx = fmaxf(fmaxf(red[0][0], red[0][1]), fmaxf(red[0][2], red[0][3]));
+	const float w = m != -INFINITY ? expf(m - mx) : 0.f; // a share without keys counts nothing
+	wz[z] = w;
+	const float ls = warp_sum(w * lz);
+	if ((z & 31) == 0) red[1][z >> 5] = ls;
+	__syncthreads();
+	if (d >= a.vd) return;
+	const float l = (red[1][0] + red[1][1]) + (red[1][2] + red[1][3]);
+	float v = 0.f;
+#pragma unroll 16
+	for (int k = 0; k < a.nsplit; ++k) v = fmaf(p[(size_t)k * pw + d], wz[k], v);
+	const float g = (a.gate ? sigmoidf_(a.gate[(size_t)n * a.ldg + (size_t)h * a.ghs + (size_t)d * a.ges]) : 1.f) / l;
+	out[((size_t)n * a.heads + h) * a.vd + d] = to_act<AT>(v * g);
+}
+
+// The same attention for decoded tokens and short portions on the warp-level tensor cores (bf16 mode): up to 16 query heads that share a
+// key/value head are the 16 rows of m16n8k16 products.  Scores and softmax weights keep fp32 accuracy: queries, keys, probabilities and
+// values enter as a bf16 value and the bf16 of what that rounding left, hi x hi + hi x lo + lo x hi summed in fp32.  One CTA per (token,
+// head tile, share of the keys); keys travel ATM_KC at a time into a double buffer of shared memory by asynchronous copies, once for
+// scores and values when the values are the first columns of the key rows (latent attention).
+#define ATM_KC 32
+#define ATM_TILES 8 // value-column tiles of 8 per warp: values up to 512 wide
+__host__ __device__ constexpr int atm_pad(int cols) { return ((cols + 15) & ~15) % 32 == 0 ? ((cols + 15) & ~15) + 8 : ((cols + 15) & ~15) + 24; } // floats per staged row: 8 mod 32, fragment reads meet 32 different banks
+__host__ __device__ constexpr int atm_ldq(int kd) { return ((kd + 15) & ~15) + 8; }
+__host__ __device__ constexpr size_t atm_smem(int kd, int vd, bool shared_kv) {
+	return (size_t)2 * ATM_KC * (atm_pad(kd) + (shared_kv ? 0 : atm_pad(vd))) * 4 + (size_t)2 * 16 * atm_ldq(kd) * 2 + (size_t)(2 * 16 * (ATM_KC + 1) + 3 * 16) * 4;
+}
+__device__ __forceinline__ void split_pair(float x, float y, uint32_t& hi, uint32_t& lo) {
+	const __nv_bfloat162 h = __floats2bfloat162_rn(x, y), l = __floats2bfloat162_rn(x - __bfloat162float(h.x), y - __bfloat162float(h.y));
+	hi = *reinterpret_cast<const uint32_t*>(&h), lo = *reinterpret_cast<const uint32_t*>(&l);
+}
+__device__ __forceinline__ void mma_bf16_16816(float (&c)[4], const uint32_t (&A)[4], const uint32_t (&B)[2]) {
+	asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+	             : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+	             : "r"(A[0]), "r"(A[1]), "r"(A[2]), "r"(A[3]), "r"(B[0]), "r"(B[1]));
+}
+__device__ __forceinline__ void cp_async4(float* dst, const float* src) {
+	asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async16(float* dst, const float* src) {
+	asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+__global__ void __launch_bounds__(256) k_seq_attn_mma(AttArgs a, bf16* out, SeqBatch sb, int shared_kv, int vec) {
+	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
+	extern __shared__ __align__(16) float sm[];
+	const int n = blockIdx.x, h0 = blockIdx.y * a.tile, R = a.tile;
+	if (a.skip && a.skip[n]) return;
+	const int kvh = h0 / a.group, kd = a.kd, vd = a.vd, kp = (kd + 15) & ~15;
+	const int ldk = atm_pad(kd), ldv = shared_kv ? ldk : atm_pad(vd), ldq = atm_ldq(kd);
+	const int kbuf = ATM_KC * ldk, vbuf = shared_kv ? 0 : ATM_KC * ldv;
+	float* const Ks = sm;                                   // [2][ATM_KC][ldk]
+	float* const Vs = shared_kv ? Ks : sm + 2 * kbuf;       // [2][ATM_KC][ldv]
+	bf16* const Qh = (bf16*)(sm + 2 * (kbuf + vbuf));       // [16][ldq]
+	bf16* const Ql = Qh + 16 * ldq;
+	float* const sc = (float*)(Ql + 16 * ldq);              // [2][16][ATM_KC + 1]: the two halves of the scores; [0]: the probabilities
+	float *const mrow = sc + 2 * 16 * (ATM_KC + 1), *const lrow = mrow + 16, *const frow = lrow + 16;
+	constexpr int LDS_ = ATM_KC + 1;
+	const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+	const int slot = sb.tslot[n], pos = sb.tpos[n];
+	int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+	if (a.chunk > 0) lo = max(lo, pos / a.chunk * a.chunk);
+	// visible keys in order: the kept first positions the window has left behind, [0, kf), then the window [lo, pos]; this CTA's share of them
+	const int kf = min(a.keep_first, lo), total = kf + pos - lo + 1;
+	const int nchunk = (total + ATM_KC - 1) / ATM_KC, per = (nchunk + a.nsplit - 1) / a.nsplit;
+	const int c_begin = (int)blockIdx.z * per, c_end = min(nchunk, c_begin + per); // chunks [c_begin, c_end)
+	auto key_pos = [&](int j) { return j < kf ? j : lo + j - kf; };
+	auto issue = [&](int c) { // one warp per key row
+		float *kb = Ks + (c & 1) * kbuf, *vb = Vs + (c & 1) * (shared_kv ? kbuf : vbuf);
+		for (int j = warp; j < ATM_KC; j += 8) {
+			const int key = c * ATM_KC + j;
+			if (key < total) {
+				const long row = cache_row(sb, slot, key_pos(key));
+				const float *ksrc = a.kc + row * a.kld + (size_t)kvh * kd, *vsrc = a.vc + row * a.vld + (size_t)kvh * vd;
+				if (vec) {
+					for (int i = 4 * lane; i < kd; i += 128) cp_async16(kb + j * ldk + i, ksrc + i);
+					if (!shared_kv)
+						for (int i = 4 * lane; i < vd; i += 128) cp_async16(vb + j * ldv + i, vsrc + i);
+				} else {
+					for (int i = lane; i < kd; i += 32) cp_async4(kb + j * ldk + i, ksrc + i);
+					if (!shared_kv)
+						for (int i = lane; i < vd; i += 32) cp_async4(vb + j * ldv + i, vsrc + i);
+				}
+				for (int i = kd + lane; i < kp; i += 32) kb[j * ldk + i] = 0.f;
+			} else { // past the last key: zeros, so that nothing read here is a NaN
+				for (int i = lane; i < kp; i += 32) kb[j * ldk + i] = 0.f;
+				if (!shared_kv)
+					for (int i = lane; i < vd; i += 32) vb[j * ldv + i] = 0.f;
+			}
 		}
-		out[((size_t)n * a.heads + h) * a.vd + d] = to_act<AT>(v * g);
+		asm volatile("cp.async.commit_group;" ::: "memory");
+	};
+	if (c_begin < c_end) issue(c_begin);
+	for (int i = tid; i < 16 * kp; i += 256) {
+		const int r = i / kp, c = i % kp;
+		const float q = r < R && c < kd ? a.q[((size_t)n * a.heads + h0 + r) * kd + c] : 0.f;
+		const bf16 hi = __float2bfloat16_rn(q);
+		Qh[r * ldq + c] = hi, Ql[r * ldq + c] = __float2bfloat16_rn(q - __bfloat162float(hi));
+	}
+	if (tid < 16) {
+		const bool sk = (a.sink || a.add_one) && blockIdx.z == 0 && tid < R; // the sink counts once: in the first share
+		mrow[tid] = sk ? (a.add_one ? 0.f : ldf(a.sink + h0 + tid)) : -INFINITY, lrow[tid] = sk ? 1.f : 0.f;
+	}
+	float acc[ATM_TILES][4];
+#pragma unroll
+	for (int i = 0; i < ATM_TILES; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+	for (int c = c_begin; c < c_end; ++c) {
+		if (c + 1 < c_end) {
+			issue(c + 1);
+			asm volatile("cp.async.wait_group 1;" ::: "memory");
+		} else asm volatile("cp.async.wait_group 0;" ::: "memory");
+		__syncthreads();
+		const float *kb = Ks + (c & 1) * kbuf, *vb = Vs + (c & 1) * (shared_kv ? kbuf : vbuf);
+		{ // scores: warp = (8 keys, every other 16 channels)
+			const int kt = warp & 3, hf = warp >> 2;
+			const float* kr = kb + (kt * 8 + g) * ldk + 2 * t;
+			const bf16 *q0 = Qh + g * ldq + 2 * t, *q1 = Ql + g * ldq + 2 * t;
+			float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f}, s2[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 3
+			for (int k0 = hf * 16; k0 < kp; k0 += 32) {
+				const float2 x = *(const float2*)(kr + k0), y = *(const float2*)(kr + k0 + 8);
+				uint32_t bh[2], bl[2];
+				split_pair(x.x, x.y, bh[0], bl[0]), split_pair(y.x, y.y, bh[1], bl[1]);
+				const uint32_t ah[4] = {*(const uint32_t*)(q0 + k0), *(const uint32_t*)(q0 + 8 * ldq + k0), *(const uint32_t*)(q0 + k0 + 8), *(const uint32_t*)(q0 + 8 * ldq + k0 + 8)};
+				const uint32_t al[4] = {*(const uint32_t*)(q1 + k0), *(const uint32_t*)(q1 + 8 * ldq + k0), *(const uint32_t*)(q1 + k0 + 8), *(const uint32_t*)(q1 + 8 * ldq + k0 + 8)};
+				mma_bf16_16816(s0, ah, bh), mma_bf16_16816(s1, ah, bl), mma_bf16_16816(s2, al, bh);
+			}
+			float* d = sc + hf * 16 * LDS_ + g * LDS_ + kt * 8 + 2 * t;
+			d[0] = s0[0] + (s1[0] + s2[0]), d[1] = s0[1] + (s1[1] + s2[1]);
+			d[8 * LDS_] = s0[2] + (s1[2] + s2[2]), d[8 * LDS_ + 1] = s0[3] + (s1[3] + s2[3]);
+		}
+		__syncthreads();
+		// softmax: two heads per warp, one key per lane
+#pragma unroll
+		for (int i = 0; i < 2; ++i) {
+			const int r = 2 * warp + i, key = c * ATM_KC + lane;
+			float s = -INFINITY;
+			if (key < total) {
+				s = (sc[r * LDS_ + lane] + sc[16 * LDS_ + r * LDS_ + lane]) * a.scale;
+				if (a.slopes && r < R) s -= a.slopes[h0 + r] * (float)(pos - key_pos(key));
+			}
+			const float mo = mrow[r], mn = fmaxf(mo, warp_max(s)), p = expf(s - mn);
+			sc[r * LDS_ + lane] = p;
+			const float ps = warp_sum(p);
+			if (lane == 0) {
+				const float f = mo == -INFINITY ? 0.f : expf(mo - mn);
+				frow[r] = f, lrow[r] = lrow[r] * f + ps, mrow[r] = mn;
+			}
+		}
+		__syncthreads();
+		// values: warp = tiles of 8 value columns; inside a 16-key step fragment places (2t, 2t+1, 2t+8, 2t+9) hold keys (t, t+4, t+8, t+12)
+		uint32_t ph[2][4], pl[2][4];
+#pragma unroll
+		for (int s = 0; s < 2; ++s) {
+			const float *p0 = sc + g * LDS_ + 16 * s + t, *p1 = p0 + 8 * LDS_;
+			split_pair(p0[0], p0[4], ph[s][0], pl[s][0]), split_pair(p1[0], p1[4], ph[s][1], pl[s][1]);
+			split_pair(p0[8], p0[12], ph[s][2], pl[s][2]), split_pair(p1[8], p1[12], ph[s][3], pl[s][3]);
+		}
+		const float f0 = frow[g], f1 = frow[g + 8];
+#pragma unroll
+		for (int i = 0; i < ATM_TILES; ++i) {
+			const int d0 = (warp + 8 * i) * 8;
+			if (d0 < vd) {
+				acc[i][0] *= f0, acc[i][1] *= f0, acc[i][2] *= f1, acc[i][3] *= f1;
+#pragma unroll
+				for (int s = 0; s < 2; ++s) {
+					const float* vp = vb + (16 * s + t) * ldv + d0 + g;
+					uint32_t bh[2], bl[2];
+					split_pair(vp[0], vp[4 * ldv], bh[0], bl[0]), split_pair(vp[8 * ldv], vp[12 * ldv], bh[1], bl[1]);
+					mma_bf16_16816(acc[i], ph[s], bh), mma_bf16_16816(acc[i], ph[s], bl), mma_bf16_16816(acc[i], pl[s], bh);
+				}
+			}
+		}
+		__syncthreads(); // this chunk's buffer may be filled again, its scores overwritten
+	}
+	if (c_begin >= c_end) __syncthreads(); // a share without keys: mrow and lrow as they were set above
+#pragma unroll
+	for (int i = 0; i < ATM_TILES; ++i)
+#pragma unroll
+		for (int e = 0; e < 4; ++e) {
+			const int r = g + (e >> 1) * 8, d = (warp + 8 * i) * 8 + 2 * t + (e & 1);
+			if (r >= R || d >= vd) continue;
+			const size_t o = (size_t)n * a.heads + h0 + r;
+			if (a.nsplit > 1) a.part[(o * a.nsplit + blockIdx.z) * (vd + 2) + d] = acc[i][e];
+			else {
+				float v = acc[i][e] / lrow[r];
+				if (a.gate) v *= sigmoidf_(a.gate[(size_t)n * a.ldg + (size_t)(h0 + r) * a.ghs + (size_t)d * a.ges]);
+				out[o * vd + d] = __float2bfloat16_rn(v);
+			}
+		}
+	if (a.nsplit > 1 && tid < R) {
+		float* p = a.part + (((size_t)n * a.heads + h0 + tid) * a.nsplit + blockIdx.z) * (vd + 2) + vd;
+		p[0] = mrow[tid], p[1] = lrow[tid];
 	}
 }
 
@@ -592,71 +780,117 @@ __global__ void k_seq_attn_gather(AttGather a, SeqBatch sb) {
 		__syncthreads();
 	}
 }
+// Which gathered columns a block of query rows sees: row t stands at position qpos0 + t; columns below kfb are the kept first positions, column
+// j >= kfb is position k0 + j - kfb.  A row's columns are [0, kept) and [lo(t), hi(t)], both ends growing with t, so what a tile of rows
+// sees is known from its first and last row: score tiles outside are not computed, and neither the softmax kernel nor the value product
+// touches 64-column blocks that no row of a 128-row tile sees.
+struct AttBand {
+	int qpos0, k0, kfb, keep_first, window, chunk;
+	__device__ __forceinline__ int lo(int t) const {
+		const int q = qpos0 + t;
+		int p = window > 0 ? max(0, q - window + 1) : 0;
+		if (chunk > 0) p = max(p, q / chunk * chunk);
+		return max(p - k0, 0) + kfb;
+	}
+	__device__ __forceinline__ int hi(int t) const { return qpos0 + t - k0 + kfb; }
+	__device__ __forceinline__ int kept() const { return max(kfb, keep_first - k0 + kfb); }
+	// does any of rows [t0, t1] see any of columns [c0, c1]?
+	__device__ __forceinline__ bool meets(int t0, int t1, int c0, int c1) const { return c0 <= hi(t1) && (c1 >= lo(t0) || c0 < kept()); }
+};
 struct AttSoftmax {
 	const float* S; // [heads of the launch][T][Cp]
 	bf16* P;        // same shape
 	int T, C, Cp;
-	int qpos0, k0, window;
-	int chunk = 0;       // > 0: a row sees only positions from floor(position / chunk) * chunk on
+	AttBand band;
+	int banded = 0;      // 1: columns outside the 64-column blocks that a 128-row tile sees are left as they are (the value product skips them)
 	const float* slopes = nullptr; // already offset to the first head of the launch, or null: score -= slopes[z] * (row position - column position)
 	int add_one = 0;     // 1: one added to the denominator
-	int keep_first, kfb; // columns below kfb are the kept first positions 0 .. kfb-1; column j >= kfb is position k0 + j - kfb
 	float scale;
 	const bf16* sink; // already offset to the first head of the launch, or null
 	const float* gate; // per head: gate[t * ldg + z], already offset to the first token and head, or null (per-channel gates are applied by the caller)
 	int ldg;
 	int split = 0;     // 1: P rows are 2 Cp wide: the probabilities as bf16, then the bf16 of what that rounding left
 };
+// One CTA per (row, head).  A thread takes pairs of neighbouring columns; the first SMX_KEEP pairs of its row stay in registers, so a row of up
+// to 512 * SMX_KEEP columns is read once.
+#define SMX_KEEP 8
 __global__ void __launch_bounds__(256) k_seq_attn_softmax(AttSoftmax a) {
 	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
-	__shared__ float red[8];
-	__shared__ float bc;
+	__shared__ float red[2][8];
 	const int t = blockIdx.x, z = blockIdx.y, tid = threadIdx.x;
 	const float* srow = a.S + ((size_t)z * a.T + t) * a.Cp;
 	bf16* prow = a.P + ((size_t)z * a.T + t) * a.Cp * (a.split ? 2 : 1);
-	const int qpos = a.qpos0 + t;
-	const int hi = min(a.C - 1, qpos - a.k0 + a.kfb); // last visible column
-	int wlo = a.window > 0 ? qpos - a.window + 1 : 0;
-	if (a.chunk > 0) wlo = max(wlo, qpos / a.chunk * a.chunk);
-	const int lo = a.kfb > 0 || a.keep_first > a.k0 ? 0 : max(0, wlo - a.k0); // nothing is visible before this column
-	auto seen = [&](int j) { // column j's position: a kept first token, or inside the window (j <= hi is the causal bound)
-		const int p = j < a.kfb ? j : a.k0 + j - a.kfb;
-		return p >= wlo || p < a.keep_first;
-	};
+	const int qpos = a.band.qpos0 + t, kfb = a.band.kfb;
+	const int lo = a.band.lo(t), hi = min(a.C - 1, a.band.hi(t)), kept = a.band.kept();
+	// columns written: everything, or the 64-column blocks that some row of this row's 128-row tile sees (a window's kept first positions: from 0 on)
+	int w0 = 0, w1 = a.Cp;
+	if (a.banded) {
+		const int t0 = t & ~127;
+		if (kept == 0) w0 = a.band.lo(t0) & ~63;
+		w1 = min(a.Cp, (a.band.hi(min(t0 + 127, a.T - 1)) | 63) + 1);
+	}
 	const float sk = a.add_one ? 0.f : a.sink ? ldf(a.sink + z) : -INFINITY;
 	const float slope = a.slopes ? a.slopes[z] : 0.f;
-	auto score = [&](int j) { return srow[j] * a.scale - slope * (float)(qpos - (j < a.kfb ? j : a.k0 + j - a.kfb)); };
+	auto score = [&](int j, float s) { // -inf for a column this row does not see
+		if (j > hi || (j < lo && j >= kept)) return -INFINITY;
+		return s * a.scale - (a.slopes ? slope * (float)(qpos - (j < kfb ? j : a.band.k0 + j - kfb)) : 0.f);
+	};
+	auto pair = [&](int j) { // j is even and Cp a multiple of 8: both columns lie inside the row
+		if (j > hi || (j + 1 < lo && j >= kept)) return make_float2(-INFINITY, -INFINITY); // nothing was computed there
+		const float2 v = *(const float2*)(srow + j);
+		return make_float2(score(j, v.x), score(j + 1, v.y));
+	};
+	float2 keep[SMX_KEEP];
 	float mx = sk;
-	for (int j = lo + tid; j <= hi; j += 256)
-		if (seen(j)) mx = fmaxf(mx, score(j));
+#pragma unroll
+	for (int i = 0; i < SMX_KEEP; ++i) {
+		if (w0 + 512 * i >= w1) break; // the row ends here (the same for the whole CTA)
+		const int j = w0 + 2 * (tid + 256 * i);
+		keep[i] = j < w1 ? pair(j) : make_float2(-INFINITY, -INFINITY);
+		mx = fmaxf(mx, fmaxf(keep[i].x, keep[i].y));
+	}
+	for (int j = w0 + 2 * (tid + 256 * SMX_KEEP); j < w1; j += 512) {
+		const float2 v = pair(j);
+		mx = fmaxf(mx, fmaxf(v.x, v.y));
+	}
 	mx = warp_max(mx);
-	if ((tid & 31) == 0) red[tid >> 5] = mx;
+	if ((tid & 31) == 0) red[0][tid >> 5] = mx;
 	__syncthreads();
-	if (tid == 0) {
-		for (int w = 1; w < 8; ++w) mx = fmaxf(mx, red[w]);
-		bc = mx;
-	}
-	__syncthreads();
-	mx = bc;
+#pragma unroll
+	for (int w = 0; w < 8; ++w) mx = fmaxf(mx, red[0][w]);
 	float sum = 0.f;
-	for (int j = lo + tid; j <= hi; j += 256)
-		if (seen(j)) sum += expf(score(j) - mx);
-	sum = warp_sum(sum);
-	__syncthreads();
-	if ((tid & 31) == 0) red[tid >> 5] = sum;
-	__syncthreads();
-	if (tid == 0) {
-		for (int w = 1; w < 8; ++w) sum += red[w];
-		if (a.sink || a.add_one) sum += expf(sk - mx);
-		bc = (a.gate ? sigmoidf_(a.gate[(size_t)t * a.ldg + z]) : 1.f) / sum;
+#pragma unroll
+	for (int i = 0; i < SMX_KEEP; ++i) {
+		if (w0 + 512 * i >= w1) break;
+		keep[i].x = expf(keep[i].x - mx), keep[i].y = expf(keep[i].y - mx);
+		sum += keep[i].x + keep[i].y;
 	}
+	for (int j = w0 + 2 * (tid + 256 * SMX_KEEP); j < w1; j += 512) {
+		const float2 v = pair(j);
+		sum += expf(v.x - mx) + expf(v.y - mx);
+	}
+	sum = warp_sum(sum);
+	if ((tid & 31) == 0) red[1][tid >> 5] = sum;
 	__syncthreads();
-	const float f = bc;
-	for (int j = tid; j < a.Cp; j += 256) {
-		const float p = j >= lo && j <= hi && seen(j) ? expf(score(j) - mx) * f : 0.f;
-		const bf16 ph = __float2bfloat16_rn(p);
-		prow[j] = ph;
-		if (a.split) prow[a.Cp + j] = __float2bfloat16_rn(p - __bfloat162float(ph));
+	sum = 0.f;
+#pragma unroll
+	for (int w = 0; w < 8; ++w) sum += red[1][w];
+	if (a.sink || a.add_one) sum += expf(sk - mx);
+	const float f = (a.gate ? sigmoidf_(a.gate[(size_t)t * a.ldg + z]) : 1.f) / sum;
+	auto put = [&](int j, float x, float y) {
+		const __nv_bfloat162 h = __floats2bfloat162_rn(x * f, y * f);
+		*(__nv_bfloat162*)(prow + j) = h;
+		if (a.split) *(__nv_bfloat162*)(prow + a.Cp + j) = __floats2bfloat162_rn(x * f - __bfloat162float(h.x), y * f - __bfloat162float(h.y));
+	};
+#pragma unroll
+	for (int i = 0; i < SMX_KEEP; ++i) {
+		if (w0 + 512 * i >= w1) break;
+		const int j = w0 + 2 * (tid + 256 * i);
+		if (j < w1) put(j, keep[i].x, keep[i].y);
+	}
+	for (int j = w0 + 2 * (tid + 256 * SMX_KEEP); j < w1; j += 512) {
+		const float2 v = pair(j);
+		put(j, expf(v.x - mx), expf(v.y - mx));
 	}
 }
 
@@ -879,12 +1113,6 @@ struct GlaArgs {
 	int heads, dim, vdim;
 	int vec;             // rows, columns and bases are 16-byte aligned: tokens are staged with 16-byte copies instead of 4-byte ones
 };
-__device__ __forceinline__ void cp_async4(float* dst, const float* src) {
-	asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp_async16(float* dst, const float* src) {
-	asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
 // One CTA of 128 threads per (sequence, head, 128 / P value columns).  The state sits in registers: P lanes share a value column,
 // each holding R of its key channels (P = 4, 8 or 16: the host takes more lanes per column when sequences x heads alone would
 // leave SMs idle, since per token a warp issues ~3 R arithmetic instructions and that, not memory, bounds a long prompt).
@@ -1251,9 +1479,9 @@ __global__ void __launch_bounds__(256) k_seq_moe_group(const int* sel, int pairs
 		}
 	}
 }
-// rows of the grouped activation matrix: Xp[row] = h[perm[row] / top]
-template <typename AT>
-__global__ void k_seq_moe_gather(AT* xp, const AT* h, const int* perm, int top, int pairs, int width) {
+// rows of the grouped activation matrix: Xp[row] = h[perm[row] / top]  (T: an element, or 16 bytes of a row; width counts in T)
+template <typename T>
+__global__ void k_seq_moe_gather(T* xp, const T* h, const int* perm, int top, int pairs, int width) {
 	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
 	const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
 	if (i >= (size_t)pairs * width) return;
@@ -1865,13 +2093,13 @@ __global__ void __launch_bounds__(64) k_seq_mingru_chunk(MinGruArgs a, SeqBatch 
 	if (ch >= a.width || (long)(k + 1) * a.chunk >= cnt) return; // the last chunk's map is not needed
 	float2* cr = a.carry + (size_t)b * a.carries * a.width + ch;
 	if (k == 0) cr[0] = make_float2(0.f, a.state[(size_t)sb.sslot[b] * a.width + ch]);
-	const float* p = a.proj + (size_t)(sb.sstart[b] + k * a.chunk) * a.ldp + ch;
+	const float* p = a.proj + (size_t)(sb.sstart[b] + k * a.chunk) * a.ldp + ch; // walks down the tokens
 	float A = 1.f, B = 0.f;
 	for (int t0 = 0; t0 < a.chunk; t0 += MINGRU_U) {
 		float zr[MINGRU_U], u[MINGRU_U];
 #pragma unroll
-		for (int i = 0; i < MINGRU_U; ++i)
-			if (t0 + i < a.chunk) zr[i] = p[(size_t)(t0 + i) * a.ldp], u[i] = p[(size_t)(t0 + i) * a.ldp + a.width];
+		for (int i = 0; i < MINGRU_U; ++i, p += a.ldp)
+			if (t0 + i < a.chunk) zr[i] = p[0], u[i] = p[a.width];
 #pragma unroll
 		for (int i = 0; i < MINGRU_U; ++i)
 			if (t0 + i < a.chunk) {
@@ -1905,18 +2133,15 @@ __global__ void __launch_bounds__(64) k_seq_mingru_apply(MinGruArgs a, AT* out, 
 	for (int t0 = 0; t0 < nt; t0 += MINGRU_U) {
 		float zr[MINGRU_U], u[MINGRU_U], g[MINGRU_U];
 #pragma unroll
-		for (int i = 0; i < MINGRU_U; ++i)
-			if (t0 + i < nt) {
-				const float* q = p + (size_t)(t0 + i) * a.ldp;
-				zr[i] = q[0], u[i] = q[a.width], g[i] = q[2 * a.width];
-			}
+		for (int i = 0; i < MINGRU_U; ++i, p += a.ldp)
+			if (t0 + i < nt) zr[i] = p[0], u[i] = p[a.width], g[i] = p[2 * a.width];
 #pragma unroll
-		for (int i = 0; i < MINGRU_U; ++i)
+		for (int i = 0; i < MINGRU_U; ++i, o += a.width)
 			if (t0 + i < nt) {
 				float keep, take;
 				mingru_step(zr[i], u[i], keep, take);
 				S = fmaf(keep, S, take);
-				o[(size_t)(t0 + i) * a.width] = to_act<AT>(S * g[i] * sigmoidf_(g[i]));
+				*o = to_act<AT>(S * g[i] * sigmoidf_(g[i]));
 			}
 	}
 	if (k * a.chunk + nt == cnt) *st = S;
@@ -1924,7 +2149,7 @@ __global__ void __launch_bounds__(64) k_seq_mingru_apply(MinGruArgs a, AT* out, 
 
 // ---------------------------------------------------------------- products  Y[n][m] = sum_k X[n][k] W[m][k]
 // blockIdx.z = batch (per-head products): X, W, Y advance by xbs, wbs, ybs elements.
-enum { EPI_F32 = 0, EPI_ACT = 1, EPI_DYT_RES = 2, EPI_RES = 3, EPI_ACT_RELU2 = 4, EPI_DECAY = 5 };
+enum { EPI_F32 = 0, EPI_ACT = 1, EPI_DYT_RES = 2, EPI_RES = 3, EPI_ACT_RELU2 = 4, EPI_DECAY = 5, EPI_SPLIT3 = 6, EPI_GLU = 7 };
 struct GemmArgs {
 	const void* X;
 	long ldx, xbs;
@@ -1935,7 +2160,9 @@ struct GemmArgs {
 	int N, M, K;
 	int epi;                 // EPI_F32: Y fp32; EPI_ACT: Y of the activation type; EPI_DYT_RES: Y fp32 residual += tanh(alpha acc) w + b;
 	                         // EPI_RES: Y fp32 residual += (res ? res : 0) + acc; EPI_ACT_RELU2: Y of the activation type = relu(acc)^2;
-	                         // EPI_DECAY: Y fp32 = sigmoid(acc)^epi_f = exp(-softplus(-acc) * epi_f)
+	                         // EPI_DECAY: Y fp32 = sigmoid(acc)^epi_f = exp(-softplus(-acc) * epi_f);
+	                         // EPI_SPLIT3: Y of the activation type, three columns `split3` apart: hi, hi, lo (value and remainder of its rounding);
+	                         // EPI_GLU: rows of W alternate gate and up, Y[n][m / 2] of the activation type = glu_unit(gate, up)
 	float epi_f;
 	const bf16 *nw, *nb, *na;
 	int w_immutable;         // W is a model weight: it may be read before the previous kernel has finished (products of gathered keys set 0)
@@ -1954,6 +2181,14 @@ struct GemmArgs {
 	const int* rs_idx = nullptr;
 	long rs_ld = 1;
 	int rs_act = 0;
+	int split3 = 0;
+	int glu_mode = 0;        // EPI_GLU: as k_seq_ff_act
+	float glu_limit = 0.f;
+	const int* x_idx = nullptr; // k_seq_gemm_skinny only: row r of X is X[x_idx[r] / x_div] (r counts from the group's first row on)
+	int x_div = 1;
+	int band_mode = 0;       // k_seq_gemm_tc only.  1: tiles of Y (rows n, columns m) that `band` does not meet are left out; 2: so are 64-deep steps of the
+	AttBand band;            // sum over k (columns of the band; with band_cp > 0 the columns are held twice, band_cp apart) that a tile's rows do not meet
+	int band_cp = 0;
 };
 // rows of batch z: first row and count
 struct GemmRows {
@@ -1980,7 +2215,10 @@ __device__ __forceinline__ void gemm_store(const GemmArgs& a, int z, const GemmR
 		return;
 	}
 	if (a.epi == EPI_F32) ((float*)a.Y)[o] = acc;
-	else if (a.epi == EPI_ACT) {
+	else if (a.epi == EPI_SPLIT3) {
+		AT* y = (AT*)a.Y + o;
+		y[0] = to_act<AT>(acc), y[a.split3] = y[0], y[2 * a.split3] = to_act<AT>(acc - ldf(y));
+	} else if (a.epi == EPI_ACT) {
 		if (a.gate) acc *= sigmoidf_(a.gate[(size_t)z * a.gbs + (size_t)(gr.base + n) * a.ldgate + m]);
 		((AT*)a.Y)[o] = to_act<AT>(acc);
 	} else if (a.epi == EPI_RES) ((float*)a.Y)[o] += a.res ? a.res[o] + acc : acc;
@@ -1989,6 +2227,19 @@ __device__ __forceinline__ void gemm_store(const GemmArgs& a, int z, const GemmR
 		const float r = fmaxf(acc, 0.f);
 		((AT*)a.Y)[o] = to_act<AT>(r * r);
 	} else ((float*)a.Y)[o] += tanhf(ldf(a.na) * acc) * ldf(a.nw + m) + ldf(a.nb + m);
+}
+
+// EPI_GLU: the pair of columns m (even: gate) and m + 1 (up)
+template <typename AT>
+__device__ __forceinline__ void gemm_store_glu(const GemmArgs& a, int z, const GemmRows& gr, int n, int m, float gate, float up) {
+	if (n >= gr.count || m >= a.M) return;
+	((AT*)a.Y)[(size_t)z * a.ybs + (size_t)(gr.base + n) * a.ldy + (m >> 1)] = to_act<AT>(glu_unit(gate, up, a.glu_limit, a.glu_mode));
+}
+// columns m (even) and m + 1 of row n
+template <typename AT>
+__device__ __forceinline__ void gemm_store2(const GemmArgs& a, int z, const GemmRows& gr, int n, int m, float x, float y) {
+	if (a.epi == EPI_GLU) gemm_store_glu<AT>(a, z, gr, n, m, x, y);
+	else gemm_store<AT>(a, z, gr, n, m, x), gemm_store<AT>(a, z, gr, n, m + 1, y);
 }
 
 // exact mode: fp32 FMA, 64 x 64 tile, 16-deep steps, 256 threads with 4 x 4 outputs each
@@ -2024,16 +2275,11 @@ __global__ void __launch_bounds__(256) k_seq_gemm_f32(GemmArgs a) {
 #pragma unroll
 	for (int i = 0; i < 4; ++i)
 #pragma unroll
-		for (int j = 0; j < 4; ++j) gemm_store<float>(a, z, gr, n0 + tn + i, m0 + tm + j, acc[i][j]);
+		for (int j = 0; j < 4; j += 2) gemm_store2<float>(a, z, gr, n0 + tn + i, m0 + tm + j, acc[i][j], acc[i][j + 1]);
 }
 
 // bf16 x bf16 -> fp32 on the tensor cores for ANY shape (edges are zero-filled in shared memory): 64 tokens x 64 rows per
 // CTA, 32-deep steps, four warps of 32 x 32.  The tcgen05 kernel below takes the shapes that fill its tiles.
-__device__ __forceinline__ void mma_bf16_16816(float (&c)[4], const uint32_t (&A)[4], const uint32_t (&B)[2]) {
-	asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-	             : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-	             : "r"(A[0]), "r"(A[1]), "r"(A[2]), "r"(A[3]), "r"(B[0]), "r"(B[1]));
-}
 #define GB_LD 40 // bf16 per shared-memory row: 32 + 8 keeps the fragment reads conflict-free
 __device__ __forceinline__ void gemm_fill_tile(bf16 (*dst)[GB_LD], const bf16* src, long ld, int r0, int rows, int k0, int K, int tid) {
 	// 64 rows x 32 columns as 256 groups of 8: two per thread
@@ -2094,8 +2340,7 @@ __global__ void __launch_bounds__(128) k_seq_gemm_bf16(GemmArgs a) {
 #pragma unroll
 		for (int j = 0; j < 4; ++j) {
 			const int n = n0 + wn + i * 16 + g, m = m0 + wm + j * 8 + 2 * t;
-			gemm_store<bf16>(a, z, gr, n, m, acc[i][j][0]), gemm_store<bf16>(a, z, gr, n, m + 1, acc[i][j][1]);
-			gemm_store<bf16>(a, z, gr, n + 8, m, acc[i][j][2]), gemm_store<bf16>(a, z, gr, n + 8, m + 1, acc[i][j][3]);
+			gemm_store2<bf16>(a, z, gr, n, m, acc[i][j][0], acc[i][j][1]), gemm_store2<bf16>(a, z, gr, n + 8, m, acc[i][j][2], acc[i][j][3]);
 		}
 }
 
@@ -2115,7 +2360,7 @@ __global__ void __launch_bounds__(NW * 32) k_seq_gemm_skinny(GemmArgs a) {
 		gr = gemm_rows(a, z);
 		if (gr.count == 0) return;
 	}
-	const bf16* X = (const bf16*)a.X + (size_t)z * a.xbs + (size_t)gr.base * a.ldx;
+	const bf16* X = (const bf16*)a.X + (size_t)z * a.xbs + (a.x_idx ? 0 : (size_t)gr.base * a.ldx);
 	const bf16* W = a.W + (size_t)z * a.wbs;
 	const bf16* w0 = W + (size_t)min(m0 + g, a.M - 1) * a.ldw;
 	const bf16* w1 = W + (size_t)min(m0 + g + 8, a.M - 1) * a.ldw;
@@ -2123,6 +2368,12 @@ __global__ void __launch_bounds__(NW * 32) k_seq_gemm_skinny(GemmArgs a) {
 	const int nslice = (a.K + 31) / 32;
 	constexpr int U = 4; // slices requested before the first is used: 8 x 16 bytes in flight per lane
 	if (!a.w_immutable && !waited) pdl_wait_prev(), waited = true;
+	long xrow[NT]; // this lane's rows of X (a routed token's own row where the rows are not grouped)
+#pragma unroll
+	for (int j = 0; j < NT; ++j) {
+		const int n = j * 8 + g;
+		xrow[j] = a.x_idx ? (n < gr.count ? (long)(a.x_idx[gr.base + n] / a.x_div) * a.ldx : 0) : (long)n * a.ldx; // x_idx comes with groups: the previous kernel has been waited for
+	}
 	for (int s0 = warp; s0 < nslice; s0 += NW * U) {
 		uint4 A0[U], A1[U];
 #pragma unroll
@@ -2140,7 +2391,7 @@ __global__ void __launch_bounds__(NW * 32) k_seq_gemm_skinny(GemmArgs a) {
 			for (int j = 0; j < NT; ++j) {
 				uint4 B = make_uint4(0, 0, 0, 0);
 				const int n = j * 8 + g;
-				if (n < gr.count && k < a.K) B = *(const uint4*)(X + (size_t)n * a.ldx + k);
+				if (n < gr.count && k < a.K) B = *(const uint4*)(X + xrow[j] + k);
 				const uint32_t B0[2] = {B.x, B.y}, B1[2] = {B.z, B.w};
 				mma_bf16_16816(acc[j], F0, B0);
 				mma_bf16_16816(acc[j], F1, B1);
@@ -2159,7 +2410,10 @@ __global__ void __launch_bounds__(NW * 32) k_seq_gemm_skinny(GemmArgs a) {
 		float v = 0.f;
 #pragma unroll
 		for (int w = 0; w < NW; ++w) v += red[w][r][n];
-		gemm_store<bf16>(a, z, gr, n, m0 + r, v);
+		if (a.epi == EPI_GLU) { // whole warps get here: 16 * NT * 8 is a multiple of 32
+			const float up = __shfl_down_sync(0xffffffffu, v, 1);
+			if (!(r & 1)) gemm_store_glu<bf16>(a, z, gr, n, m0 + r, v, up);
+		} else gemm_store<bf16>(a, z, gr, n, m0 + r, v);
 	}
 }
 

@@ -95,7 +95,7 @@ struct Seq {
 	void *hA = nullptr, *a1 = nullptr, *a2 = nullptr; // activation type (float or bf16)
 	size_t w_proj = 0, w_f = 0, w_a = 0;              // widths (elements per token)
 	// prompt attention as products: gathered keys / transposed values of one key head, scores and probabilities
-	bool attn_products = true;
+	bool attn_products = true, attn_mma = true;
 	bf16 *att_kb = nullptr, *att_vt = nullptr, *att_p = nullptr;
 	float* att_s = nullptr;
 	size_t cap_kb = 0, cap_vt = 0, cap_sp = 0;
@@ -318,6 +318,8 @@ void validate(const Seq& s) {
 		if (!sandwich && (L.dwa || m.res_gate)) CALM_FATAL("seq: layer %d: depth average and residual gate are served in sandwich blocks", i);
 		if (sandwich && (!L.norm1.w || !L.norm1b.w || (L.ff > 0 && (!L.norm2.w || !L.norm2b.w)))) CALM_FATAL("seq: layer %d: sandwich blocks have a norm before and after every sublayer", i);
 		if (sandwich && m.res_gate && L.ff > 0 && (L.ff_kind == SEQ_FF_MOE) == (L.w_rg2 != nullptr)) CALM_FATAL("seq: layer %d: the feed-forward's residual gate rides with the router's rows, or is w_rg2", i);
+		if (L.glu_rows && (L.ff <= 0 || L.ff_kind == SEQ_FF_RELU2 || (L.ff_kind == SEQ_FF_MOE && (L.expert_act == 1 || m.block == SEQ_BLOCK_HYPER))))
+			CALM_FATAL("seq: layer %d: glu_rows is an option of gated units (of routed experts outside hyper blocks)", i);
 		if (L.ff > 0) {
 			if (L.ff_kind < SEQ_FF_CLAMPED || L.ff_kind > SEQ_FF_GATED) CALM_FATAL("seq: layer %d: unknown feed-forward kind %d", i, L.ff_kind);
 			if (L.ff_kind == SEQ_FF_GATED && L.ff_act != SEQ_ACT_SILU && L.ff_act != SEQ_ACT_GELU_TANH) CALM_FATAL("seq: layer %d: unknown activation %d", i, L.ff_act);
@@ -432,7 +434,19 @@ struct GemmExtra {
 	const int* rs_idx = nullptr;
 	long rs_ld = 1;
 	int rs_act = 0;
+	int split3 = 0;              // EPI_SPLIT3: columns between the three copies
+	int glu_mode = 0;            // EPI_GLU
+	float glu_limit = 0.f;
+	const int* x_idx = nullptr;  // grouped product read through an index (gemm_skinny_fits says whether it may be given)
+	int x_div = 1;
+	int band_mode = 0, band_cp = 0; // products of attention: what a band of visible columns leaves out
+	AttBand band = {};
 };
+bool al8(long v) { return v % 8 == 0; }
+// products of few rows that the weight-streaming kernel takes
+bool gemm_skinny_fits(const Seq& s, const void* X, long ldx, long xbs, const void* W, long ldw, long wbs, int N, int K) {
+	return !s.m.exact && N <= 32 && al8(K) && al8(ldx) && al8(ldw) && al8(xbs) && al8(wbs) && ((uintptr_t)X & 15) == 0 && ((uintptr_t)W & 15) == 0;
+}
 void gemm(Seq& s, const void* X, long ldx, long xbs, const void* W, long ldw, long wbs, void* Y, long ldy, long ybs, int N, int M, int K, int batch, int epi,
           const SeqNorm* nrm = nullptr, int kind_as = -1, bool w_immutable = true, const GemmExtra* ex = nullptr) {
 	GemmArgs a;
@@ -440,6 +454,7 @@ void gemm(Seq& s, const void* X, long ldx, long xbs, const void* W, long ldw, lo
 	if (!ex) ex = &none;
 	a.bias = (const bf16*)ex->bias, a.res = ex->res, a.gate = ex->gate, a.ldgate = ex->ldgate, a.gbs = ex->gbs, a.seg = ex->seg, a.x_rows = ex->x_rows, a.epi_f = ex->epi_f, a.split = ex->split, a.split_act = ex->split_act, a.Y2 = ex->Y2, a.ldy2 = ex->ldy2, a.out_scale = ex->out_scale;
 	a.rs = ex->rs, a.rs_idx = ex->rs_idx, a.rs_ld = ex->rs_ld, a.rs_act = ex->rs_act;
+	a.split3 = ex->split3, a.glu_mode = ex->glu_mode, a.glu_limit = ex->glu_limit, a.x_idx = ex->x_idx, a.x_div = ex->x_div, a.band_mode = ex->band_mode, a.band_cp = ex->band_cp, a.band = ex->band;
 	a.w_immutable = w_immutable;
 	a.X = X, a.ldx = ldx, a.xbs = xbs, a.W = (const bf16*)W, a.ldw = ldw, a.wbs = wbs, a.Y = Y, a.ldy = ldy, a.ybs = ybs;
 	a.N = N, a.M = M, a.K = K, a.epi = epi;
@@ -447,14 +462,14 @@ void gemm(Seq& s, const void* X, long ldx, long xbs, const void* W, long ldw, lo
 	// a grouped product does the work of its x_rows rows, and reads at most that many groups' weights
 	const double rows = ex->seg ? (double)ex->x_rows : (double)N * batch, mats = ex->seg ? std::min((double)batch, rows) : (double)batch;
 	const double flops = 2.0 * rows * M * K;
-	const double bytes = mats * M * K * 2 + rows * K * act_size(s) + rows * M * 4;
+	const double bytes = mats * M * K * 2 + rows * K * act_size(s) + rows * M * (epi == EPI_GLU ? act_size(s) / 2.0 : epi == EPI_ACT || epi == EPI_ACT_RELU2 ? (double)act_size(s) : epi == EPI_SPLIT3 ? 6.0 : 4.0);
 	if (s.tc && gemm_tc_fits(a, batch)) {
 		bool launched = false;
-		run_kernel(s, kind_as >= 0 ? kind_as : KD_GEMM_TC, bytes, flops, [&] { launched = gemm_tc_launch(a, batch, s.stream); });
+		run_kernel(s, kind_as >= 0 ? kind_as : KD_GEMM_TC, bytes, flops, [&] { launched = gemm_tc_launch(a, batch, s.stream, s.pdl); });
 		if (launched) return;
 	}
-	auto al8 = [](long v) { return v % 8 == 0; };
-	if (!s.m.exact && N <= 32 && K % 8 == 0 && al8(ldx) && al8(ldw) && al8(xbs) && al8(wbs) && ((uintptr_t)X & 15) == 0 && ((uintptr_t)W & 15) == 0) {
+	if (a.band_mode == 2) CALM_FATAL("seq: a banded value product needs the tcgen05 kernel"); // what the band leaves out of its input was never written
+	if (gemm_skinny_fits(s, X, ldx, xbs, W, ldw, wbs, N, K)) {
 		const dim3 grid(cdiv(M, 16), 1, batch);
 		const bool few = (long)cdiv(M, 16) * batch < 3L * s.sms && K >= 1024; // few CTAs: twice the warps per CTA keep as many bytes in flight
 		run_kernel(s, kind_as >= 0 ? kind_as : KD_GEMM_SKINNY, bytes, flops, [&] {
@@ -470,6 +485,7 @@ void gemm(Seq& s, const void* X, long ldx, long xbs, const void* W, long ldw, lo
 		});
 		return;
 	}
+	if (a.x_idx) CALM_FATAL("seq: rows through an index are read by the weight-streaming kernel only");
 	const dim3 grid(cdiv(M, 64), cdiv(N, 64), batch);
 	run_kernel(s, kind_as >= 0 ? kind_as : KD_GEMM, bytes, flops, [&] {
 		if (s.m.exact) launch_k(s, k_seq_gemm_f32, grid, 256, 0, a);
@@ -511,10 +527,36 @@ void hc_read(Seq& s, void* out, const int* rows, const void* in, const SeqNorm& 
 		else launch_k(s, k_seq_hc_read<bf16>, R, threads, 0, (bf16*)out, s.x, rows, (const bf16*)in, (const bf16*)nm.w, wl, s.m.norm_offset, s.m.eps, R, W, S);
 	});
 }
-// CTAs that share the keys of one (token, head tile): few tokens over a long context
-int attn_nsplit(const Seq& s, int live_tokens, int tiles, int window, int longest) {
-	const int ctas = live_tokens * tiles, chunks = cdiv(window > 0 ? std::min(longest, window) : longest, ATT_KC);
-	return ctas >= 2 * s.sms ? 1 : std::max(1, std::min({chunks, 2 * s.sms / ctas, 128}));
+// How a step's short portions and decoded tokens run through attention: query heads per CTA and CTAs that share the keys of one (token,
+// head tile) when few tokens look back over a long context.  bf16 mode takes the tensor-core kernel wherever its shared memory and registers
+// hold the heads' width.
+struct AttnPlan {
+	bool mma;
+	int tile, nsplit;
+	size_t smem;
+};
+// shares of the keys, rounded up to a few values per octave: a decode graph is captured once per value, not once per chunk that a context grows by
+int round_split(int n) {
+	int v = 1;
+	while (v < n) v = v < 4 ? v + 1 : (v & (v - 1)) ? v / 3 * 4 : v / 2 * 3; // 1 2 3 4 6 8 12 16 24 ...
+	return v;
+}
+AttnPlan attn_plan(const Seq& s, int group, int kd, int vd, bool shared_kv, int heads, int live_tokens, int span, int longest) {
+	AttnPlan p;
+	p.smem = atm_smem(kd, vd, shared_kv);
+	p.mma = s.attn_mma && !s.m.exact && p.smem <= 220 * 1024 && vd <= 8 * 8 * ATM_TILES;
+	const int keys = span > 0 ? std::min(longest, span) : longest;
+	if (p.mma) {
+		p.tile = std::min(group, 16);
+		while (group % p.tile) --p.tile;
+		const int ctas = live_tokens * (heads / p.tile), room = s.sms * std::max(1, std::min(4, (int)(227 * 1024 / (p.smem + 1024))));
+		p.nsplit = ctas >= room ? 1 : std::max(1, std::min({round_split(cdiv(keys, ATM_KC)), room / ctas, ATT_MAXSPLIT}));
+	} else {
+		p.tile = attn_tile(group, kd, vd), p.smem = attn_smem(p.tile, kd);
+		const int ctas = live_tokens * (heads / p.tile);
+		p.nsplit = ctas >= 2 * s.sms ? 1 : std::max(1, std::min({round_split(cdiv(keys, ATT_KC)), 2 * s.sms / ctas, ATT_MAXSPLIT}));
+	}
+	return p;
 }
 void ensure_carry(Seq& s, size_t need) {
 	if (need <= s.carry_cap) return;
@@ -559,7 +601,7 @@ void attention_products(Seq& s, int kind, const AttArgs& a, bf16* out, const Seq
 		int k0 = a.window > 0 ? std::max(0, q0 - a.window + 1) : 0;
 		if (a.chunk > 0) k0 = std::max(k0, q0 / a.chunk * a.chunk); // the first query's block; later rows mask what lies before theirs
 		const int kfb = a.window > 0 ? std::min(a.keep_first, k0) : 0;
-		const int C = kfb + q0 + Tb - k0, Cp = (C + 7) & ~7;
+		const int C = kfb + q0 + Tb - k0, Cp = (C + 63) & ~63; // whole 64-deep steps of the value product
 		// split: queries [hi | hi | lo] against keys [hi | lo | hi] (depth 3 kd), probabilities [hi | lo] against the values held twice (depth Cp + C)
 		const int sx = a.split ? 3 : 1, px = a.split ? 2 : 1;
 		reserve_attn(s, (size_t)C * a.kd * sx, (size_t)a.vd * Cp * px, (size_t)a.group * Tb * Cp * px);
@@ -570,29 +612,38 @@ void attention_products(Seq& s, int kind, const AttArgs& a, bf16* out, const Seq
 			run_kernel(s, kind, (double)C * (a.kd + a.vd) * (4 + 2 * sx), 0, [&] { launch_k(s, k_seq_attn_gather, dim3(cdiv(Cp, 32), 4), 256, 0, g, sb); });
 			const int h0 = kvh * a.group;
 			const bf16* q = (const bf16*)s.a3 + ((size_t)(first + t0) * a.heads + h0) * a.kd * sx;
-			gemm(s, q, (long)a.heads * a.kd * sx, a.kd * sx, s.att_kb, a.kd * sx, 0, s.att_s, Cp, (long)Tb * Cp, Tb, C, a.kd * sx, a.group, EPI_F32, nullptr, kind, false);
+			const AttBand band{q0, k0, kfb, a.window > 0 ? a.keep_first : 0, a.window, a.chunk};
+			GemmExtra sx_band, gx;
+			sx_band.band_mode = 1, sx_band.band = band;
+			bf16* const o = out + ((size_t)(first + t0) * a.heads + h0) * a.vd;
+			// value product: only where the tcgen05 kernel takes it are the columns that a tile of rows does not see left out
+			GemmArgs pv;
+			pv.X = s.att_p, pv.ldx = (long)Cp * px, pv.xbs = (long)Tb * Cp * px, pv.W = s.att_vt, pv.ldw = (long)Cp * px, pv.wbs = 0, pv.N = Tb, pv.M = a.vd, pv.K = a.split ? Cp + C : C, pv.seg = nullptr;
+			const CUtensorMap *mw, *mx;
+			const bool banded = s.tc && gemm_tc_fits(pv, a.group) && gemm_tc_maps(pv, a.group, mw, mx);
+			if (banded) gx.band_mode = 2, gx.band = band, gx.band_cp = a.split ? Cp : 0;
+			gemm(s, q, (long)a.heads * a.kd * sx, a.kd * sx, s.att_kb, a.kd * sx, 0, s.att_s, Cp, (long)Tb * Cp, Tb, C, a.kd * sx, a.group, EPI_F32, nullptr, kind, false, &sx_band);
 			AttSoftmax sm;
-			sm.S = s.att_s, sm.P = s.att_p, sm.T = Tb, sm.C = C, sm.Cp = Cp, sm.qpos0 = q0, sm.k0 = k0, sm.window = a.window, sm.scale = a.scale;
-			sm.keep_first = a.window > 0 ? a.keep_first : 0, sm.kfb = kfb, sm.split = a.split;
-			sm.chunk = a.chunk, sm.slopes = a.slopes ? a.slopes + h0 : nullptr, sm.add_one = a.add_one;
+			sm.S = s.att_s, sm.P = s.att_p, sm.T = Tb, sm.C = C, sm.Cp = Cp, sm.scale = a.scale, sm.band = band, sm.banded = banded, sm.split = a.split;
+			sm.slopes = a.slopes ? a.slopes + h0 : nullptr, sm.add_one = a.add_one;
 			const bool head_gate = a.gate && a.ges == 0; // one gate per head scales the probabilities; a gate per channel goes into the value product's epilogue
 			sm.sink = a.sink ? a.sink + h0 : nullptr, sm.gate = head_gate ? a.gate + (size_t)(first + t0) * a.ldg + h0 : nullptr, sm.ldg = a.ldg;
-			GemmExtra gx;
 			if (a.gate && !head_gate) gx.gate = a.gate + (size_t)(first + t0) * a.ldg + (size_t)h0 * a.ghs, gx.ldgate = a.ldg, gx.gbs = a.ghs;
 			run_kernel(s, kind, (double)a.group * Tb * Cp * (4 + 2 * px), 0, [&] { launch_k(s, k_seq_attn_softmax, dim3(Tb, a.group), 256, 0, sm); });
-			gemm(s, s.att_p, (long)Cp * px, (long)Tb * Cp * px, s.att_vt, (long)Cp * px, 0, out + ((size_t)(first + t0) * a.heads + h0) * a.vd, (long)a.heads * a.vd, a.vd, Tb, a.vd,
-			     a.split ? Cp + C : C, a.group, EPI_ACT, nullptr, kind, false, &gx);
+			gemm(s, s.att_p, pv.ldx, pv.xbs, s.att_vt, pv.ldw, 0, o, (long)a.heads * a.vd, a.vd, Tb, a.vd, pv.K, a.group, EPI_ACT, nullptr, kind, false, &gx);
 		}
 		t0 += Tb;
 	}
 }
 
-void attention(Seq& s, int kind, AttArgs a, void* out, const SeqBatch& sb, double kv_rows, int longest) {
+// q_ready: the queries already wait in a3, in the form the product path reads
+void attention(Seq& s, int kind, AttArgs a, void* out, const SeqBatch& sb, double kv_rows, int longest, bool q_ready = false) {
 	a.skip = nullptr;
 	bool rest = true;
 	if (!s.m.exact && s.attn_products && s.n_on_products > 0) {
 		const size_t n = (size_t)sb.N * a.heads * a.kd;
-		if (a.split) run_kernel(s, KD_ELEMENT, n * 10.0, 0, [&] { launch_k(s, k_seq_split_q, cdiv(n, 256), 256, 0, (bf16*)s.a3, a.q, a.kd, (size_t)sb.N * a.heads); });
+		if (q_ready) {
+		} else if (a.split) run_kernel(s, KD_ELEMENT, n * 10.0, 0, [&] { launch_k(s, k_seq_split_q, cdiv(n, 256), 256, 0, (bf16*)s.a3, a.q, a.kd, (size_t)sb.N * a.heads); });
 		else run_kernel(s, KD_ELEMENT, n * 6.0, 0, [&] { launch_k(s, k_seq_cast_cols<bf16>, cdiv(n, 256), 256, 0, (bf16*)s.a3, a.q, a.heads * a.kd, 0, a.heads * a.kd, sb.N); });
 		for (int b = 0; b < sb.B; ++b)
 			if (s.hb_count[b] >= kAttnGemmMin) attention_products(s, kind, a, (bf16*)out, sb, s.hb_slot[b], s.hb_start[b], s.hb_count[b], s.hb_pos0[b]);
@@ -600,25 +651,28 @@ void attention(Seq& s, int kind, AttArgs a, void* out, const SeqBatch& sb, doubl
 		rest = s.n_on_products < sb.B;
 	}
 	if (!rest) return;
-	const size_t smem = attn_smem(a.tile, a.kd);
-	// few tokens over a long context: the keys of one (token, head tile) are shared out over several CTAs
-	const int live = a.skip ? std::max(1, sb.N - s.tok_on_products) : sb.N; // tokens the fused kernel really serves (the others' CTAs leave at once)
+	const int live = a.skip ? std::max(1, sb.N - s.tok_on_products) : sb.N; // tokens served here (the others' CTAs leave at once)
 	int span = a.window > 0 ? a.window + a.keep_first : 0;
 	if (a.chunk > 0) span = span > 0 ? std::min(span, a.chunk) : a.chunk;
-	a.nsplit = attn_nsplit(s, live, a.heads / a.tile, span, longest);
+	const bool shared_kv = a.kc == a.vc;
+	const AttnPlan p = attn_plan(s, a.group, a.kd, a.vd, shared_kv, a.heads, live, span, longest);
+	a.tile = p.tile, a.nsplit = p.nsplit;
 	ensure_part(s, (size_t)sb.N * a.heads * a.nsplit * (a.vd + 2));
 	a.part = s.part;
 	const dim3 grid(sb.N, a.heads / a.tile, a.nsplit);
-	const double bytes = kv_rows * (a.heads / a.group) * (a.kc == a.vc ? a.kd : a.kd + a.vd) * 4.0;
+	const double bytes = kv_rows * (a.heads / a.group) * (shared_kv ? a.kd : a.kd + a.vd) * 4.0;
 	const double flops = 2.0 * kv_rows * a.heads * (a.kd + a.vd);
 	run_kernel(s, kind, a.skip ? 0 : bytes, a.skip ? 0 : flops, [&] {
-		if (s.m.exact) launch_k(s, k_seq_attention<float>, grid, ATT_THREADS, smem, a, (float*)out, sb);
-		else launch_k(s, k_seq_attention<bf16>, grid, ATT_THREADS, smem, a, (bf16*)out, sb);
+		auto al4 = [](long v) { return v % 4 == 0; };
+		if (p.mma) launch_k(s, k_seq_attn_mma, grid, 256, p.smem, a, (bf16*)out, sb, shared_kv ? 1 : 0, al4(a.kd) && al4(a.kld) && (shared_kv || (al4(a.vd) && al4(a.vld))) ? 1 : 0);
+		else if (s.m.exact) launch_k(s, k_seq_attention<float>, grid, ATT_THREADS, p.smem, a, (float*)out, sb);
+		else launch_k(s, k_seq_attention<bf16>, grid, ATT_THREADS, p.smem, a, (bf16*)out, sb);
 	});
 	if (a.nsplit > 1)
 		run_kernel(s, kind, 0, 0, [&] {
-			if (s.m.exact) launch_k(s, k_seq_attention_merge<float>, dim3(sb.N, a.heads), 128, 0, a, (float*)out);
-			else launch_k(s, k_seq_attention_merge<bf16>, dim3(sb.N, a.heads), 128, 0, a, (bf16*)out);
+			const dim3 mg(sb.N, a.heads, cdiv(a.vd, 128));
+			if (s.m.exact) launch_k(s, k_seq_attention_merge<float>, mg, 128, 0, a, (float*)out);
+			else launch_k(s, k_seq_attention_merge<bf16>, mg, 128, 0, a, (bf16*)out);
 		});
 }
 
@@ -743,15 +797,23 @@ void mixer_typed(Seq& s, const SeqLayer& L, RunState& r, const SeqBatch& sb, dou
 			GemmExtra ux;
 			ux.split = H * Pr, ux.split_act = 1, ux.Y2 = a2, ux.ldy2 = (long)H * D;
 			gemm(s, a1, Rq, 0, L.w_uq, Rq, 0, s.f[1], (long)H * Pr, 0, N, H * (Pr + D), Rq, 1, EPI_F32, nullptr, -1, true, &ux);
-			run_kernel(s, KD_QK, (double)N * H * Pr * 8, 0, [&] { launch_k(s, k_seq_rope_heads, N, 128, (Pr / 2) * sizeof(float2), s.f[0], s.f[1], H, (long)H * kd, kd, Rk, rope, sb); });
 		} else gemm(s, a1, Rq, 0, L.w_uq, Rq, 0, a2, (long)H * D, 0, N, H * D, Rq, 1, EPI_ACT);
-		// the key up-projection moves to the query side: q'_h = W_uk,h^T q_h, so scores and values are taken on the cached latent itself
-		gemm(s, a2, (long)H * D, D, L.w_ukT, D, (long)Rk * D, s.f[0], (long)H * kd, kd, N, Rk, D, H, EPI_F32);
+		// the key up-projection moves to the query side: q'_h = W_uk,h^T q_h, so scores and values are taken on the cached latent itself.  When all of
+		// the step's attention runs as products the queries go straight to the matrix those read: rounded, or as value and remainder
+		const bool direct = !s.m.exact && s.attn_products && s.n_on_products == sb.B;
+		const int kq = direct && L.scores_f32 ? 3 * kd : kd, split3 = direct && L.scores_f32 ? kd : 0;
+		if (Pr > 0)
+			run_kernel(s, KD_QK, (double)N * H * Pr * (direct ? 4 + 2 * (split3 ? 3 : 1) : 8), 0, [&] {
+				launch_k(s, k_seq_rope_heads, N, 128, (Pr / 2) * sizeof(float2), s.f[0], direct ? (bf16*)s.a3 : nullptr, split3, s.f[1], H, (long)H * kq, kq, Rk, rope, sb);
+			});
+		GemmExtra qx;
+		qx.split3 = split3;
+		gemm(s, a2, (long)H * D, D, L.w_ukT, D, (long)Rk * D, direct ? s.a3 : (void*)s.f[0], (long)H * kq, kq, N, Rk, D, H, split3 ? EPI_SPLIT3 : direct ? EPI_ACT : EPI_F32, nullptr, -1, true, &qx);
 		AttArgs a;
-		a.q = s.f[0], a.kc = a.vc = r.cache_a, a.kld = a.vld = kd, a.heads = H, a.group = H, a.tile = attn_tile(H, kd, Rk), a.kd = kd, a.vd = Rk, a.window = L.window;
+		a.q = s.f[0], a.kc = a.vc = r.cache_a, a.kld = a.vld = kd, a.heads = H, a.group = H, a.kd = kd, a.vd = Rk, a.window = L.window;
 		a.scale = L.scale, a.sink = (const bf16*)L.sink, a.gate = L.no_gate ? nullptr : proj + Rq + (own ? kd : 0), a.ldg = P, a.ghs = 1, a.ges = 0, a.keep_first = 0;
 		a.split = L.scores_f32;
-		attention(s, KD_ATTN_LATENT, a, a1, sb, L.window > 0 ? std::min(kv_rows, (double)N * L.window) : kv_rows, longest);
+		attention(s, KD_ATTN_LATENT, a, a1, sb, L.window > 0 ? std::min(kv_rows, (double)N * L.window) : kv_rows, longest, direct);
 		gemm(s, a1, (long)H * Rk, Rk, L.w_uv, Rk, (long)Dv * Rk, a2, (long)H * Dv, Dv, N, Dv, Rk, H, EPI_ACT);
 		out_product<AT>(s, a2, L.w_o, N, H * Dv, oe, L.b_o);
 	} else if (L.type == SEQ_MINGRU) {
@@ -760,7 +822,7 @@ void mixer_typed(Seq& s, const SeqLayer& L, RunState& r, const SeqBatch& sb, dou
 		for (int b = 0; b < sb.B; ++b) most = std::max(most, s.hb_count[b]);
 		MinGruArgs g;
 		g.proj = proj, g.ldp = P, g.width = D, g.state = r.delta;
-		g.chunk = std::max(64, cdiv(most, 64)); // at most 64 maps to fold
+		g.chunk = std::max(32, cdiv(most, 64)); // 32 tokens measured fastest on 2048-token prompts; at most 64 maps to fold
 		const int chunks = cdiv(most, g.chunk);
 		g.carries = chunks;
 		if (chunks > 1) ensure_carry(s, (size_t)sb.B * chunks * D);
@@ -810,7 +872,7 @@ void mixer_typed(Seq& s, const SeqLayer& L, RunState& r, const SeqBatch& sb, dou
 		const size_t qk_smem = ((size_t)2 * std::max(L.rot_dims / 2, 1) + H + G) * sizeof(float);
 		run_kernel(s, KD_QK, (double)N * (H * D + G * D + G * Dv) * 8, 0, [&] { launch_k(s, k_seq_qk_rope, N, 256, qk_smem, qa, sb); });
 		AttArgs a;
-		a.q = s.f[0], a.kc = r.cache_a, a.vc = r.cache_b, a.kld = G * D, a.vld = G * Dv, a.heads = H, a.group = H / G, a.tile = attn_tile(H / G, D, Dv), a.kd = D, a.vd = Dv;
+		a.q = s.f[0], a.kc = r.cache_a, a.vc = r.cache_b, a.kld = G * D, a.vld = G * Dv, a.heads = H, a.group = H / G, a.kd = D, a.vd = Dv;
 		a.window = L.window, a.keep_first = L.window > 0 ? L.keep_first : 0, a.scale = L.scale, a.sink = nullptr;
 		a.gate = L.no_gate ? nullptr : proj + H * D + G * D + G * Dv, a.ldg = P, a.ghs = L.gate_per_head ? 1 : Dv, a.ges = L.gate_per_head ? 0 : 1; // a sigmoid gate per output channel (or per head), from the same stacked projection
 		a.chunk = L.chunk, a.slopes = L.dist_bias ? r.slopes : nullptr, a.add_one = L.add_one;
@@ -902,7 +964,7 @@ void mixer_typed(Seq& s, const SeqLayer& L, RunState& r, const SeqBatch& sb, dou
 		ca.seg[2] = ConvSeg{H * D + G * D, G, Dv, 0, 0, 1.f, 1, r.cache_b};
 		conv(s, L, r, ca, sb, proj, P);
 		AttArgs a;
-		a.q = s.f[0], a.kc = r.cache_a, a.vc = r.cache_b, a.kld = G * D, a.vld = G * Dv, a.heads = H, a.group = H / G, a.tile = attn_tile(H / G, D, Dv), a.kd = D, a.vd = Dv;
+		a.q = s.f[0], a.kc = r.cache_a, a.vc = r.cache_b, a.kld = G * D, a.vld = G * Dv, a.heads = H, a.group = H / G, a.kd = D, a.vd = Dv;
 		a.window = L.window, a.scale = L.scale, a.sink = (const bf16*)L.sink, a.gate = nullptr, a.ldg = 0, a.ghs = 1, a.ges = 0, a.keep_first = 0;
 		attention(s, KD_ATTN_WINDOW, a, a2, sb, L.window > 0 ? std::min(kv_rows, (double)N * L.window) : kv_rows, longest);
 		out_product<AT>(s, a2, L.w_o, N, H * Dv, oe, L.b_o);
@@ -914,6 +976,14 @@ template <typename AT>
 void feed_forward(Seq& s, const SeqLayer& L, const SeqBatch& sb, const OutEpi& oe) {
 	const int N = sb.N, W = s.m.width;
 	AT *hA = (AT*)s.hA, *a2 = (AT*)s.a2;
+	// rows of w_gate_up that alternate gate and up: the unit leaves the product's epilogue in the activation type
+	GemmExtra glu;
+	glu.glu_limit = L.limit, glu.glu_mode = L.ff_kind == SEQ_FF_CLAMPED || (L.ff_kind == SEQ_FF_MOE && L.expert_act == 2) ? 0 : L.ff_kind == SEQ_FF_GATED && L.ff_act == SEQ_ACT_GELU_TANH ? 2 : 1;
+	if (L.glu_rows && L.ff_kind != SEQ_FF_MOE) {
+		gemm(s, hA, W, 0, L.w_gate_up, W, 0, a2, L.ff, 0, N, 2 * L.ff, W, 1, EPI_GLU, nullptr, -1, true, &glu);
+		out_product<AT>(s, a2, L.w_down, N, L.ff, oe);
+		return;
+	}
 	if (L.ff_kind == SEQ_FF_CLAMPED) {
 		gemm(s, hA, W, 0, L.w_gate_up, W, 0, s.proj, 2L * L.ff, 0, N, 2 * L.ff, W, 1, EPI_F32);
 		run_kernel(s, KD_ELEMENT, (double)N * L.ff * (8 + sizeof(AT)), 0,
@@ -971,8 +1041,14 @@ void feed_forward(Seq& s, const SeqLayer& L, const SeqBatch& sb, const OutEpi& o
 			           [&] { launch_k(s, k_seq_moe_route, cdiv(N, 4), 128, 0, logits, ldl, Et, top, N, s.moe_sel, s.moe_wt, L.route_mode, (const bf16*)L.correction, rscale); });
 			run_kernel(s, KD_ROUTE, (double)pairs * 4 * Et, 0, [&] { launch_k(s, k_seq_moe_group, Et, 256, 0, s.moe_sel, pairs, Et, s.moe_seg, s.moe_perm, s.moe_inv); });
 		}
-		run_kernel(s, KD_ELEMENT, (double)pairs * W * 2 * sizeof(AT), 0,
-		           [&] { launch_k(s, k_seq_moe_gather<AT>, cdiv((long)pairs * W, 256), 256, 0, (AT*)s.moe_x, hA, s.moe_perm, top, pairs, W); });
+		// few rows: the products read a pair's token through the index; many: the pairs' rows are gathered first
+		const bool indexed = L.glu_rows && gemm_skinny_fits(s, hA, W, 0, L.w_gate_up, W, 2L * ff * W, N, W);
+		if (!indexed)
+			run_kernel(s, KD_ELEMENT, (double)pairs * W * 2 * sizeof(AT), 0, [&] {
+				const size_t row = (size_t)W * sizeof(AT);
+				if (row % 16 == 0) launch_k(s, k_seq_moe_gather<uint4>, cdiv(pairs * (row / 16), 256), 256, 0, (uint4*)s.moe_x, (const uint4*)hA, s.moe_perm, top, pairs, (int)(row / 16));
+				else launch_k(s, k_seq_moe_gather<AT>, cdiv((long)pairs * W, 256), 256, 0, (AT*)s.moe_x, hA, s.moe_perm, top, pairs, W);
+			});
 		GemmExtra gx;
 		gx.seg = s.moe_seg, gx.x_rows = pairs;
 		if (r2) {
@@ -991,7 +1067,11 @@ void feed_forward(Seq& s, const SeqLayer& L, const SeqBatch& sb, const OutEpi& o
 			post_norm<AT>(s, sf > 0 ? s.mo : nullptr, HcMoe{s.moe_d, s.moe_inv, s.moe_sel, L.weight_input ? nullptr : s.moe_wt, top, E}, *oe.post, N);
 			return;
 		}
-		gemm(s, s.moe_x, W, 0, L.w_gate_up, W, 2L * ff * W, s.moe_y, 2L * ff, 0, N, 2 * ff, W, E, EPI_F32, nullptr, -1, true, &gx);
+		if (L.glu_rows) {
+			glu.seg = s.moe_seg, glu.x_rows = pairs;
+			if (indexed) glu.x_idx = s.moe_perm, glu.x_div = top;
+			gemm(s, indexed ? (const void*)hA : s.moe_x, W, 0, L.w_gate_up, W, 2L * ff * W, s.moe_a, ff, 0, N, 2 * ff, W, E, EPI_GLU, nullptr, -1, true, &glu);
+		} else gemm(s, s.moe_x, W, 0, L.w_gate_up, W, 2L * ff * W, s.moe_y, 2L * ff, 0, N, 2 * ff, W, E, EPI_F32, nullptr, -1, true, &gx);
 		if (oe.hc) {
 			// hyper blocks: the shared unit's product is the base of y, the routed sum is formed while the streams are written; the two units'
 			// activations are one launch
@@ -1008,8 +1088,9 @@ void feed_forward(Seq& s, const SeqLayer& L, const SeqBatch& sb, const OutEpi& o
 			hc_write<AT>(s, *oe.hc, sf > 0 ? s.mo : nullptr, HcMoe{s.moe_d, s.moe_inv, s.moe_sel, s.moe_wt, top, E}, N, oe.next_in, oe.next_norm);
 			return;
 		}
-		run_kernel(s, KD_ELEMENT, (double)pairs * ff * (8 + sizeof(AT)), 0,
-		           [&] { launch_k(s, k_seq_ff_act<AT>, cdiv((long)pairs * ff, 256), 256, 0, (AT*)s.moe_a, s.moe_y, ff, pairs, L.limit, L.expert_act == 2 ? 0 : 1, 2 * ff); });
+		if (!L.glu_rows)
+			run_kernel(s, KD_ELEMENT, (double)pairs * ff * (8 + sizeof(AT)), 0,
+			           [&] { launch_k(s, k_seq_ff_act<AT>, cdiv((long)pairs * ff, 256), 256, 0, (AT*)s.moe_a, s.moe_y, ff, pairs, L.limit, L.expert_act == 2 ? 0 : 1, 2 * ff); });
 		gemm(s, s.moe_a, ff, 0, L.w_down, ff, (long)W * ff, s.moe_d, W, 0, N, W, ff, E, EPI_F32, nullptr, -1, true, &gx);
 		if (oe.sand) { // sandwich blocks: the weighted sum is formed by the kernel that gates and norms it
 			Sandwich a = *oe.sand;
@@ -1161,7 +1242,7 @@ void forward_decode_graph(Seq& s, const SeqBatch& sb, int n_want, double kv_rows
 		if (L.type != SEQ_LATENT && L.type != SEQ_WINDOW && L.type != SEQ_GQA) return; // recurrent mixers: nothing to share out
 		const bool lat = L.type == SEQ_LATENT;
 		const int group = lat ? L.heads : L.heads / L.kv_heads, kd = lat ? L.kv_rank + L.rot_dims : L.dim, vd = lat ? L.kv_rank : L.vdim;
-		const int ns = attn_nsplit(s, sb.N, L.heads / attn_tile(group, kd, vd), attn_span(L), longest);
+		const int ns = attn_plan(s, group, kd, vd, lat, L.heads, sb.N, attn_span(L), longest).nsplit;
 		key.push_back(ns);
 		part_need = std::max(part_need, (size_t)sb.N * L.heads * ns * (vd + 2));
 	};
@@ -1227,6 +1308,7 @@ extern "C" void* calm_b200_seq_prepare(const struct SeqModel* model) {
 	for (cudaEvent_t& e : s.ev) CUDA_CHECK(cudaEventCreate(&e));
 	for (cudaEvent_t& e : s.timer) CUDA_CHECK(cudaEventCreate(&e));
 	if (const char* e = getenv("CALM_B200_SEQ_ATTN_PRODUCTS")) s.attn_products = atoi(e) != 0;
+	if (const char* e = getenv("CALM_B200_SEQ_ATTN_MMA")) s.attn_mma = atoi(e) != 0;
 	if (const char* e = getenv("CALM_B200_SEQ_GRAPH")) s.use_graph = atoi(e) != 0;
 	if (const char* e = getenv("CALM_B200_SEQ_PDL")) s.pdl = atoi(e) != 0;
 	const char* tc = getenv("CALM_B200_SEQ_TC");
@@ -1304,6 +1386,7 @@ extern "C" void* calm_b200_seq_prepare(const struct SeqModel* model) {
 		constexpr int R = decltype(r)::value, P = decltype(p)::value;
 		CUDA_CHECK(cudaFuncSetAttribute(k_seq_gla_scan<R, P>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)gla_smem(R, P)));
 	});
+	CUDA_CHECK(cudaFuncSetAttribute(k_seq_attn_mma, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
 	CUDA_CHECK(cudaFuncSetAttribute(k_seq_attention<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024));
 	CUDA_CHECK(cudaFuncSetAttribute(k_seq_attention<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024));
 	// rotation tables of the grouped-query and latent attentions: angle step per rotated pair (in double), rescaled between two wavelengths

@@ -112,8 +112,12 @@ def plan(cfg: dict, tensors: Dict[str, torch.Tensor]) -> Tuple[dict, List[dict],
                        norm2=need(p + "norm2", [width]), norm2b=need(p + "norm2b", [width]))
             rec["w_router"] = stack(f + "in", [need(p + "rg2", [width, width]), need(f + "router", [E, width])])
             rec["b_router"] = biases(f + "in.b", [(p + "rg2.b", width), ("", E)])
-            # experts side by side: [experts][gate | up] and [experts][down], so that one grouped product serves all of them
-            rec["w_gate_up"] = stack(f + "gate_ups", [need(f + f"e{e}.{n}", [ff, width]) for e in range(E) for n in ("gate", "up")])
+            # experts side by side, [experts][gate and up rows alternating] and [experts][down]: one grouped product serves all of them, and the unit is
+            # formed in its epilogue
+            rec["glu_rows"] = 1
+            pairs = [torch.stack([up.pop(need(f + f"e{e}.{n}", [ff, width])) for n in ("gate", "up")], 1).reshape(2 * ff, width) for e in range(E)]
+            up[f + "gate_ups"] = torch.cat(pairs, 0).contiguous()
+            rec["w_gate_up"] = f + "gate_ups"
             rec["w_down"] = stack(f + "downs", [need(f + f"e{e}.down", [width, ff]) for e in range(E)])
         layers.append(rec)
     head = {"vocab": vocab, "width": width, "eps": float(cfg["norm"]["eps"]), "embed": need("embed", [vocab, width]), "head": "embed",

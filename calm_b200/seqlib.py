@@ -46,7 +46,7 @@ SeqLayer._fields_ = [(n, C.c_int) for n in ("type", "heads", "kv_heads", "dim", 
                                                                          ("w_sh_gate_up", C.c_void_p), ("w_sh_down", C.c_void_p),
                                                                          ("qk_per_head", C.c_int), ("gate_per_head", C.c_int), ("b_o", C.c_void_p), ("scores_f32", C.c_int), ("ff_act", C.c_int),
                                                                          ("expert_act", C.c_int), ("weight_input", C.c_int), ("shared_gate", C.c_int), ("kv_shared", C.c_int),
-                                                                         ("dwa", C.c_void_p), ("w_rg2", C.c_void_p), ("b_rg2", C.c_void_p)]
+                                                                         ("dwa", C.c_void_p), ("w_rg2", C.c_void_p), ("b_rg2", C.c_void_p)] + [("glu_rows", C.c_int)]
 
 
 class SeqModel(C.Structure):

@@ -208,6 +208,8 @@ struct SeqLayer {
 	const void* dwa;       /* bf16 [layer index + 2]: weights of the depth average, or NULL: the stream goes on as it is */
 	const void* w_rg2;     /* res_gate, feed-forward other than SEQ_FF_MOE: (width, width) and bf16 [width] or NULL */
 	const void* b_rg2;
+	/* gated units */
+	int glu_rows;          /* 1: the rows of w_gate_up alternate gate and up (row 2c gate c, row 2c + 1 up c), the unit is formed in the product's epilogue */
 };
 
 struct SeqModel {

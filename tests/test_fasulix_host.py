@@ -40,7 +40,7 @@ def test_plan_binds_every_size_from_the_config():
     assert torch.equal(up[a["b_in"]][24:44], t["l0.mix.z.b"]) and torch.equal(up[a["b_in"]][44:64], t["l0.mix.x.b"]) and not up[a["b_in"]][64:].any()
     assert a["ff_kind"] == seqlib.FF_MOE and a["route_mode"] == 1 and a["expert_act"] == 2 and a["limit"] == 0.8 and a["experts"] == 3 and a["top"] == 2
     assert up[a["w_router"]].shape == (27, 24) and torch.equal(up[a["w_router"]][24:], t["l0.mlp.router"]) and torch.equal(up[a["b_router"]][:24], t["l0.rg2.b"]) and not up[a["b_router"]][24:].any()
-    assert up[a["w_gate_up"]].shape == (3 * 24, 24) and torch.equal(up[a["w_gate_up"]][24:36], t["l0.mlp.e1.gate"]) and torch.equal(up[a["w_gate_up"]][36:48], t["l0.mlp.e1.up"])
+    assert up[a["w_gate_up"]].shape == (3 * 24, 24) and torch.equal(up[a["w_gate_up"]][24:48:2], t["l0.mlp.e1.gate"]) and torch.equal(up[a["w_gate_up"]][25:48:2], t["l0.mlp.e1.up"])
     assert up[a["w_down"]].shape == (72, 12) and up[a["dwa"]].shape == (2,)
     assert b["type"] == seqlib.SEQ_LATENT and b["no_gate"] == 1 and b["rot_dims"] == 4 and b["rot_base"] == 100.0 and "window" not in b and up[b["sink"]].shape == (3,)
     assert up[b["w_in"]].shape == (24 + 10 + 18, 24) and "ff" not in b and "norm2" not in b and up[b["dwa"]].shape == (3,)
@@ -97,9 +97,9 @@ def test_records_match_the_header():
     text = open(os.path.join(root, "include", "calm_b200_seq.h")).read()
     body = text[text.index("struct SeqLayer {"):text.index("struct SeqModel {")]
     names = [n for n, _ in seqlib.SeqLayer._fields_]
-    tail = ["kv_shared", "dwa", "w_rg2", "b_rg2"]
+    tail = ["kv_shared", "dwa", "w_rg2", "b_rg2", "glu_rows"]
     assert names[-len(tail):] == tail
-    at = [body.index((" " if n == "kv_shared" else "* ") + n + ";") for n in tail]
+    at = [body.index((" " if n in ("kv_shared", "glu_rows") else "* ") + n + ";") for n in tail]
     assert at == sorted(at)
     assert [n for n, _ in seqlib.SeqModel._fields_][-2:] == ["logit_scale", "res_gate"]
     model = text[text.index("struct SeqModel {"):]
