@@ -142,14 +142,14 @@ struct PairRope {
 	const double* freq; // [dims / 2]
 	float mag;
 };
-__device__ __forceinline__ float2 rope_pair(const PairRope& r, int pos, int i, float u, float v) {
-	double sd, cd;
-	sincos((double)pos * r.freq[i], &sd, &cd);
-	const float c = (float)cd * r.mag, s = (float)sd * r.mag;
-	return make_float2(u * c - v * s, v * c + u * s);
+__device__ __forceinline__ float2 rope_angle(const PairRope& r, int pos, int i) { // (cos, sin) of pair i
+	double s, c;
+	sincos((double)pos * r.freq[i], &s, &c);
+	return make_float2((float)c * r.mag, (float)s * r.mag);
 }
+__device__ __forceinline__ float2 rope_turn(float2 cs, float u, float v) { return make_float2(u * cs.x - v * cs.y, v * cs.x + u * cs.y); }
 template <typename AT>
-__global__ void k_seq_latent_norm(const float* proj, int ldp, RmsSeg sq, RmsSeg sc, AT* cq, float* cache, PairRope rope, SeqBatch sb, float eps) {
+__global__ void k_seq_latent_norm(const float* proj, int ldp, RmsSeg sq, RmsSeg sc, AT* cq, float* cache, PairRope rope, float2* cs, SeqBatch sb, float eps) {
 	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
 	const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 	const int n = blockIdx.x * (blockDim.x >> 5) + warp;
@@ -163,43 +163,39 @@ __global__ void k_seq_latent_norm(const float* proj, int ldp, RmsSeg sq, RmsSeg 
 	if (blockIdx.y == 0) {
 		AT* d = cq + (size_t)n * s.len;
 		for (int i = lane; i < s.len; i += 32) d[i] = to_act<AT>(src[i] * r * ldf(s.w + i));
+		for (int i = lane; i < rope.dims / 2; i += 32) cs[(size_t)n * (rope.dims / 2) + i] = rope_angle(rope, sb.tpos[n], i); // for the queries of this layer
 	} else {
 		const int pos = sb.tpos[n];
 		float* d = cache + cache_row(sb, sb.tslot[n], pos) * (s.len + rope.dims);
 		for (int i = lane; i < s.len; i += 32) d[i] = src[i] * r * ldf(s.w + i);
 		for (int i = lane; i < rope.dims / 2; i += 32) {
-			const float2 t = rope_pair(rope, pos, i, src[s.len + 2 * i], src[s.len + 2 * i + 1]);
+			const float2 t = rope_turn(rope_angle(rope, pos, i), src[s.len + 2 * i], src[s.len + 2 * i + 1]);
 			d[s.len + 2 * i] = t.x, d[s.len + 2 * i + 1] = t.y;
 		}
 	}
 }
-// the rotated query channels of every head: q[n][h * ldh + col + d] from src [N][heads * dims]; one CTA per token, the angles are formed once.
-// qb given: the queries leave in the activation type instead (split3 = 0), or as [hi | hi | lo] rows of split3 columns each (see k_seq_split_q).
-__global__ void __launch_bounds__(128) k_seq_rope_heads(float* q, bf16* qb, int split3, const float* src, int heads, long ldq, int ldh, int col, PairRope rope, SeqBatch sb) {
+// the rotated query channels of every head: q[n][h * ldh + col + d] from src [N][heads * dims], cs [N][dims / 2] the angles k_seq_latent_norm
+// formed.  qb given: the queries leave in the activation type instead (split3 = 0), or as [hi | hi | lo] rows of split3 columns each (see
+// k_seq_split_q).  One thread per pair.
+__global__ void __launch_bounds__(256) k_seq_rope_heads(float* q, bf16* qb, int split3, const float* src, const float2* cs, int heads, int dims, long ldq, int ldh, int col, int N) {
 	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
-	extern __shared__ float2 cs2[]; // [dims / 2] (cos, sin)
-	const int n = blockIdx.x, half = rope.dims / 2;
-	for (int i = threadIdx.x; i < half; i += blockDim.x) {
-		double s, c;
-		sincos((double)sb.tpos[n] * rope.freq[i], &s, &c);
-		cs2[i] = make_float2((float)c * rope.mag, (float)s * rope.mag);
+	const int half = dims / 2;
+	const size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+	if (e >= (size_t)N * heads * half) return;
+	const size_t n = e / (heads * half);
+	const int h = (int)(e % (heads * half)) / half, i = (int)(e % half);
+	const float2 uv = *(const float2*)(src + 2 * e), r = rope_turn(cs[n * half + i], uv.x, uv.y);
+	const size_t o = n * ldq + (size_t)h * ldh + col + 2 * i;
+	if (!qb) {
+		q[o] = r.x, q[o + 1] = r.y;
+		return;
 	}
-	__syncthreads();
-	for (int e = threadIdx.x; e < heads * half; e += blockDim.x) {
-		const int h = e / half, i = e % half;
-		const float u = src[(size_t)n * heads * rope.dims + 2 * e], v = src[(size_t)n * heads * rope.dims + 2 * e + 1];
-		const float r0 = u * cs2[i].x - v * cs2[i].y, r1 = v * cs2[i].x + u * cs2[i].y;
-		if (!qb) {
-			float* d = q + (size_t)n * ldq + (size_t)h * ldh + col + 2 * i;
-			d[0] = r0, d[1] = r1;
-			continue;
-		}
-		bf16* d = qb + (size_t)n * ldq + (size_t)h * ldh + col + 2 * i;
-		d[0] = __float2bfloat16_rn(r0), d[1] = __float2bfloat16_rn(r1);
-		if (split3 > 0) {
-			d[split3] = d[0], d[split3 + 1] = d[1];
-			d[2 * split3] = __float2bfloat16_rn(r0 - __bfloat162float(d[0])), d[2 * split3 + 1] = __float2bfloat16_rn(r1 - __bfloat162float(d[1]));
-		}
+	const bf16 h0 = __float2bfloat16_rn(r.x), h1 = __float2bfloat16_rn(r.y);
+	bf16* d = qb + o;
+	d[0] = h0, d[1] = h1;
+	if (split3 > 0) {
+		d[split3] = h0, d[split3 + 1] = h1;
+		d[2 * split3] = __float2bfloat16_rn(r.x - __bfloat162float(h0)), d[2 * split3 + 1] = __float2bfloat16_rn(r.y - __bfloat162float(h1));
 	}
 }
 
@@ -360,8 +356,19 @@ struct AttArgs {
 	const int* skip;  // [N] or null: 1 = this token's attention is computed by the product path (k_seq_attn_*), the CTA leaves
 	int nsplit;       // CTAs that share one (token, head tile)'s keys; > 1: partial results go to `part`, k_seq_attention_merge finishes
 	float* part;      // [N][heads][nsplit][vd + 2]: unnormalised output, running maximum, denominator
+	const float* qr = nullptr;  // the last `rot` query channels of every head come from here instead, [N][heads * rot], and are turned by the angles in cs
+	const float2* cs = nullptr; // [N][rot / 2]
+	int rot = 0;
 	int split = 0;    // 1: on the product path queries, keys and probabilities travel as bf16 pairs (value + remainder), so scores and weights keep fp32 accuracy
 };
+// channel c of the query of (token, head)
+__device__ __forceinline__ float att_query(const AttArgs& a, int n, int h, int c) {
+	const int e = c - (a.kd - a.rot);
+	if (!a.qr || e < 0) return a.q[((size_t)n * a.heads + h) * a.kd + c];
+	const float* p = a.qr + ((size_t)n * a.heads + h) * a.rot + (e & ~1);
+	const float2 r = rope_turn(a.cs[(size_t)n * (a.rot / 2) + e / 2], p[0], p[1]);
+	return e & 1 ? r.y : r.x;
+}
 template <typename AT>
 __global__ void __launch_bounds__(ATT_THREADS) k_seq_attention(AttArgs a, AT* out, SeqBatch sb) {
 	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
@@ -385,7 +392,7 @@ __global__ void __launch_bounds__(ATT_THREADS) k_seq_attention(AttArgs a, AT* ou
 	// this CTA's share of the key chunks (the whole range when nsplit == 1)
 	const int nchunk = (total + ATT_KC - 1) / ATT_KC, per = (nchunk + a.nsplit - 1) / a.nsplit;
 	const int c_begin = (int)blockIdx.z * per * ATT_KC, c_end = min(total - 1, ((int)blockIdx.z + 1) * per * ATT_KC - 1);
-	for (int i = tid; i < R * a.kd; i += ATT_THREADS) qs[i] = a.q[((size_t)n * a.heads + h0) * a.kd + i];
+	for (int i = tid; i < R * a.kd; i += ATT_THREADS) qs[i] = att_query(a, n, h0 + i / a.kd, i % a.kd);
 	if (tid < R) {
 		const bool sk = (a.sink || a.add_one) && blockIdx.z == 0; // the sink counts once: in the first share
 		mrow[tid] = sk ? (a.add_one ? 0.f : ldf(a.sink + h0 + tid)) : -INFINITY, lrow[tid] = sk ? 1.f : 0.f;
@@ -628,11 +635,24 @@ __global__ void __launch_bounds__(256) k_seq_attn_mma(AttArgs a, bf16* out, SeqB
 		asm volatile("cp.async.commit_group;" ::: "memory");
 	};
 	if (c_begin < c_end) issue(c_begin);
-	for (int i = tid; i < 16 * kp; i += 256) {
-		const int r = i / kp, c = i % kp;
-		const float q = r < R && c < kd ? a.q[((size_t)n * a.heads + h0 + r) * kd + c] : 0.f;
-		const bf16 hi = __float2bfloat16_rn(q);
-		Qh[r * ldq + c] = hi, Ql[r * ldq + c] = __float2bfloat16_rn(q - __bfloat162float(hi));
+	const int kq = a.qr ? kd - a.rot : kd; // channels read as they are; the rest are turned here
+	for (int r = warp; r < 16; r += 8) { // one warp per query row
+		bf16 *qh = Qh + r * ldq, *ql = Ql + r * ldq;
+		const float* qsrc = a.q + ((size_t)n * a.heads + h0 + r) * kd;
+		auto put = [&](int c, float q) {
+			const bf16 hi = __float2bfloat16_rn(q);
+			qh[c] = hi, ql[c] = __float2bfloat16_rn(q - __bfloat162float(hi));
+		};
+		if (r < R) {
+#pragma unroll 8
+			for (int c = lane; c < kq; c += 32) put(c, qsrc[c]);
+			for (int i = lane; i < (kd - kq) / 2; i += 32) {
+				const float* p = a.qr + ((size_t)n * a.heads + h0 + r) * a.rot + 2 * i;
+				const float2 v = rope_turn(a.cs[(size_t)n * (a.rot / 2) + i], p[0], p[1]);
+				put(kq + 2 * i, v.x), put(kq + 2 * i + 1, v.y);
+			}
+		}
+		for (int c = (r < R ? kd : 0) + lane; c < kp; c += 32) put(c, 0.f);
 	}
 	if (tid < 16) {
 		const bool sk = (a.sink || a.add_one) && blockIdx.z == 0 && tid < R; // the sink counts once: in the first share

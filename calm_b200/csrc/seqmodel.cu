@@ -75,6 +75,8 @@ struct Seq {
 	float *x = nullptr, *x0 = nullptr, *proj = nullptr, *f[6] = {};
 	float* hist = nullptr;                            // depth average: X_0 (the embedding rows), X_1 .. X_layers of the step's tokens, [layers + 1][N][width]
 	bool depth = false;                               // some layer averages over depth
+	float2* rope_cs = nullptr;                        // SEQ_LATENT: cos and sin of the layer's rotated pairs, [N][rot_dims / 2]
+	size_t w_rope = 0;
 	float2* carry = nullptr;                          // SEQ_MINGRU: chunk maps of a step's longer portions
 	size_t carry_cap = 0;
 	void* ah = nullptr;                               // parallel blocks: a dense unit's hidden activations, written by the mixer's input product
@@ -398,6 +400,7 @@ void reserve_tokens(Seq& s, int N, int B, int W) {
 		}
 		s.x = (float*)dalloc(cn * s.streams * s.m.width * sizeof(float));
 		s.x0 = (float*)dalloc(cn * s.m.width * sizeof(float));
+		if (s.w_rope) cudaFree(s.rope_cs), s.rope_cs = (float2*)dalloc(cn * s.w_rope * sizeof(float2));
 		if (s.depth) cudaFree(s.hist), s.hist = (float*)dalloc((s.layers.size() + 1) * cn * s.m.width * sizeof(float));
 		s.proj = (float*)dalloc(cn * s.w_proj * sizeof(float));
 		for (float*& p : s.f) p = (float*)dalloc(cn * s.w_f * sizeof(float));
@@ -792,7 +795,7 @@ void mixer_typed(Seq& s, const SeqLayer& L, RunState& r, const SeqBatch& sb, dou
 		const PairRope rope{Pr, rt == s.rot.end() ? nullptr : rt->second.first, rt == s.rot.end() ? 1.f : rt->second.second};
 		const bool own = !L.kv_shared; // a layer that reads another one's cache has only its query latent to norm
 		run_kernel(s, KD_NORM, (double)N * (Rq + (own ? kd : 0)) * 8, 0,
-		           [&] { launch_k(s, k_seq_latent_norm<AT>, dim3(cdiv(N, 4), own ? 2 : 1), 128, 0, proj, P, sq, sc, a1, r.cache_a, rope, sb, s.m.eps); });
+		           [&] { launch_k(s, k_seq_latent_norm<AT>, dim3(cdiv(N, 4), own ? 2 : 1), 128, 0, proj, P, sq, sc, a1, r.cache_a, rope, s.rope_cs, sb, s.m.eps); });
 		if (Pr > 0) { // one product for both parts of the queries: the rotated channels stay fp32, the others leave in the activation type
 			GemmExtra ux;
 			ux.split = H * Pr, ux.split_act = 1, ux.Y2 = a2, ux.ldy2 = (long)H * D;
@@ -802,9 +805,11 @@ void mixer_typed(Seq& s, const SeqLayer& L, RunState& r, const SeqBatch& sb, dou
 		// the step's attention runs as products the queries go straight to the matrix those read: rounded, or as value and remainder
 		const bool direct = !s.m.exact && s.attn_products && s.n_on_products == sb.B;
 		const int kq = direct && L.scores_f32 ? 3 * kd : kd, split3 = direct && L.scores_f32 ? kd : 0;
-		if (Pr > 0)
+		// otherwise the attention kernel turns the rotated channels as it reads them, unless the product path needs them too
+		const bool turned = !direct && (s.m.exact || !s.attn_products || s.n_on_products == 0);
+		if (Pr > 0 && !turned)
 			run_kernel(s, KD_QK, (double)N * H * Pr * (direct ? 4 + 2 * (split3 ? 3 : 1) : 8), 0, [&] {
-				launch_k(s, k_seq_rope_heads, N, 128, (Pr / 2) * sizeof(float2), s.f[0], direct ? (bf16*)s.a3 : nullptr, split3, s.f[1], H, (long)H * kq, kq, Rk, rope, sb);
+				launch_k(s, k_seq_rope_heads, cdiv((long)N * H * Pr / 2, 256), 256, 0, s.f[0], direct ? (bf16*)s.a3 : nullptr, split3, s.f[1], s.rope_cs, H, Pr, (long)H * kq, kq, Rk, N);
 			});
 		GemmExtra qx;
 		qx.split3 = split3;
@@ -813,6 +818,7 @@ void mixer_typed(Seq& s, const SeqLayer& L, RunState& r, const SeqBatch& sb, dou
 		a.q = s.f[0], a.kc = a.vc = r.cache_a, a.kld = a.vld = kd, a.heads = H, a.group = H, a.kd = kd, a.vd = Rk, a.window = L.window;
 		a.scale = L.scale, a.sink = (const bf16*)L.sink, a.gate = L.no_gate ? nullptr : proj + Rq + (own ? kd : 0), a.ldg = P, a.ghs = 1, a.ges = 0, a.keep_first = 0;
 		a.split = L.scores_f32;
+		if (turned && Pr > 0) a.qr = s.f[1], a.cs = s.rope_cs, a.rot = Pr;
 		attention(s, KD_ATTN_LATENT, a, a1, sb, L.window > 0 ? std::min(kv_rows, (double)N * L.window) : kv_rows, longest, direct);
 		gemm(s, a1, (long)H * Rk, Rk, L.w_uv, Rk, (long)Dv * Rk, a2, (long)H * Dv, Dv, N, Dv, Rk, H, EPI_ACT);
 		out_product<AT>(s, a2, L.w_o, N, H * Dv, oe, L.b_o);
@@ -1441,6 +1447,7 @@ extern "C" void* calm_b200_seq_prepare(const struct SeqModel* model) {
 		if (L.w_rg2) s.w_fsh = std::max(s.w_fsh, (size_t)m.width);
 		if (L.ff > 0 && L.ff_kind == SEQ_FF_RELU2 && L.in_tail > 0) s.w_ah = std::max(s.w_ah, (size_t)L.ff);
 		size_t wf = 0, wa = (size_t)L.ff;
+		if (L.type == SEQ_LATENT) s.w_rope = std::max(s.w_rope, (size_t)L.rot_dims / 2);
 		if (L.type == SEQ_LATENT) wf = (size_t)L.heads * (L.kv_rank + L.rot_dims), wa = std::max({wa, (size_t)L.heads * (L.kv_rank + L.rot_dims) * (L.scores_f32 ? 3 : 1), (size_t)L.heads * L.dim, (size_t)L.heads * L.vdim, (size_t)L.q_rank});
 		if (L.type == SEQ_DELTA) wf = std::max((size_t)L.heads * L.dim, (size_t)L.heads * L.vdim), wa = std::max({wa, (size_t)L.heads * L.vdim, (size_t)L.a_rank + L.g_rank});
 		if (L.type == SEQ_MINGRU) wa = std::max(wa, (size_t)L.dim);
@@ -1469,7 +1476,7 @@ extern "C" void calm_b200_seq_release(void* handle) {
 		for (RunState& q : r.sub) drop(q);
 	};
 	for (RunState& r : s->runs) drop(r);
-	cudaFree(s->lin), cudaFree(s->fsh), cudaFree(s->hist), cudaFree(s->carry);
+	cudaFree(s->lin), cudaFree(s->fsh), cudaFree(s->hist), cudaFree(s->carry), cudaFree(s->rope_cs);
 	cudaFree(s->table_dev), cudaFree(s->d_tok), cudaFree(s->d_want), cudaFree(s->d_argmax), cudaFree(s->logits), cudaFree(s->hW);
 	cudaFree(s->part), cudaFree(s->a3), cudaFree(s->att_kb), cudaFree(s->att_vt), cudaFree(s->att_s), cudaFree(s->att_p), cudaFree(s->x), cudaFree(s->x0), cudaFree(s->proj), cudaFree(s->hA), cudaFree(s->a1), cudaFree(s->a2), cudaFree(s->trace_buf);
 	for (float* p : s->f) cudaFree(p);
