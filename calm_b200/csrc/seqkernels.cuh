@@ -755,7 +755,7 @@ __global__ void __launch_bounds__(256) k_seq_attn_mma(AttArgs a, bf16* out, SeqB
 // For many query tokens of one sequence the scores and the weighted values are matrix products on the tensor cores:
 // the keys of the visible range are gathered from the paged cache into a bf16 matrix (values transposed), S = Q K^T per
 // head, a row-wise fp32 softmax applies scale, causal / window mask, sink and output gate and writes bf16 probabilities,
-// then O = P V.  k_seq_attention above serves single decoded tokens, short portions and the exact mode.
+// then O = P V.  Single decoded tokens and short portions take k_seq_attn_mma above, the exact mode k_seq_attention.
 struct AttGather {
 	const float* kc;
 	const float* vc;

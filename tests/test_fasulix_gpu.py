@@ -19,7 +19,7 @@ import fasulix_plain as plain  # noqa: E402
 
 pytestmark = pytest.mark.gpu
 
-from calm_b200 import container, fasulix, registry, serving  # noqa: E402
+from calm_b200 import container, fasulix, registry, seqlib, serving  # noqa: E402
 
 
 def moe(experts=5, top=2, ff=12, limit=0.9):
@@ -403,6 +403,46 @@ def test_prompt_attention_as_products_keeps_the_scores_exact(monkeypatch):
                 wrong = copy.deepcopy(cfg)
                 wrong["layers"][0]["mixer"]["mask"]["size"] += off
                 assert rel_err(plain.forward(wrong, as_f64(t), toks), ref) > 4 * errs["1"]
+
+
+def test_decode_attention_on_tensor_cores_keeps_the_scores_exact(monkeypatch):
+    """bfloat16 mode serves decoded tokens and short portions with a tensor-core kernel whose scores, weights and values enter as bf16 value +
+    remainder: with sharp scores it stays as close to the plain statement as the fused fp32 kernel it replaces.  Seventeen heads make two
+    head tiles, 40 keys more than one staged chunk, a latent width that is no multiple of 16 or 4 the unaligned copies."""
+    for kw in (dict(heads=17, kv_rank=40, rot_dim=8), dict(heads=16, kv_rank=37, rot_dim=2, vdim=5), dict(heads=3, kv_rank=64, rot_dim=16)):
+        cfg = config([latent(scale=1.5, **kw), latent(size=37, scale=1.5, kv_from=0, **kw)])
+        t, toks = weights(cfg, 19), tokens(cfg, 90)
+        t["l0.mix.sink"] += 1.0
+        ref = plain.forward(cfg, as_f64(t), toks)
+        errs = {}
+        for mma in ("1", "0"):
+            monkeypatch.setenv("CALM_B200_SEQ_ATTN_MMA", mma)
+            with fasulix.from_tensors(cfg, t, "bfloat16", max_tokens=300, max_seqs=2, page=8) as m:
+                errs[mma] = max(rel_err(in_portions(m, toks, cut), ref, "bfloat16") for cut in ([1], [15, 7], [80, 1]))
+        assert errs["1"] < TOL["bfloat16"] and errs["0"] < TOL["bfloat16"] and errs["1"] < 1.5 * errs["0"] + 1e-3
+
+
+@pytest.mark.parametrize("alternate", [1, 0])
+def test_dense_units_in_sandwich_blocks(alternate):
+    """A feed-forward of one routed expert weighs it by one, so the same weights bound as a dense clamped unit (its rows alternating or
+    stacked, the residual gate a matrix of its own) must give the same logits."""
+    cfg = config([gru(mlp=moe(experts=1, top=1, ff=20)), latent(size=5, mlp=moe(experts=1, top=1, ff=9))])
+    t, toks = weights(cfg, 20), tokens(cfg, 33)
+    ref = plain.forward(cfg, as_f64(t), toks)
+    head, layers, up = fasulix.plan(cfg, t)
+    W = cfg["width"]
+    for i, rec in enumerate(layers):
+        f = f"l{i}.mlp."
+        up[f + "rg2"], up[f + "rg2.b"] = up[rec["w_router"]][:W].contiguous(), up[rec["b_router"]][:W].contiguous()
+        if not alternate:
+            up[rec["w_gate_up"]] = torch.cat([up[rec["w_gate_up"]][0::2], up[rec["w_gate_up"]][1::2]], 0).contiguous()
+        for k in ("w_router", "b_router", "experts", "top", "route_mode", "route_scale", "expert_act"):
+            del rec[k]
+        rec.update(ff_kind=seqlib.FF_CLAMPED, glu_rows=alternate, w_rg2=f + "rg2", b_rg2=f + "rg2.b")
+    for dtype in ("float32", "bfloat16"):
+        with seqlib.SeqDeviceModel(head, layers, up, exact=dtype == "float32", max_tokens=128, max_seqs=2, page=8) as m:
+            for cut in ([33], [20, 1]):
+                assert rel_err(in_portions(m, toks, cut), ref, dtype) < TOL[dtype]
 
 
 def test_tensor_core_products_match_the_warp_level_ones(monkeypatch):
