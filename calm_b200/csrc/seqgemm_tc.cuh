@@ -42,6 +42,7 @@ __device__ __forceinline__ bool mbar_wait_bounded(uint64_t* bar, uint32_t parity
 // of the plain ones -- a bias at most, and for EPI_F32 columns past `split` in the activation type -- with everything that does not depend on
 // the token worked out before the loop; TG_ANY: gemm_store decides per element.
 #define TG_ANY (-1)
+#define TG_ACT_GATE 100 // EPI_ACT times sigmoid(gate)
 template <int E>
 __device__ __forceinline__ void tg_epilogue(const GemmArgs& a, int z, const GemmRows& gr, int n0, int m, int lane, uint32_t tmem) {
 	const int rows = min(TG_BN, gr.count - n0);
@@ -52,6 +53,8 @@ __device__ __forceinline__ void tg_epilogue(const GemmArgs& a, int z, const Gemm
 	const size_t o = aside ? (size_t)(gr.base + n0) * a.ldy2 + (m - a.split) : (size_t)z * a.ybs + (size_t)(gr.base + n0) * a.ldy + (E == EPI_GLU ? m >> 1 : m);
 	float* const yf = (float*)a.Y + o;
 	bf16* const yb = (bf16*)(aside ? a.Y2 : a.Y) + o;
+	const float* gate = E == TG_ACT_GATE ? a.gate + (size_t)z * a.gbs + (size_t)(gr.base + n0) * a.ldgate + m : nullptr; // advances with the row pointer
+	const size_t gstep = E == TG_ACT_GATE ? a.ldgate : 0;
 	for (int c0 = 0; c0 < rows; c0 += 32) {
 		float v[32];
 		tmem_ld32(tmem + c0, v);
@@ -74,13 +77,14 @@ __device__ __forceinline__ void tg_epilogue(const GemmArgs& a, int z, const Gemm
 				}
 			} else {
 #pragma unroll
-				for (int j = 0; j < 32; ++j, q += step) {
+				for (int j = 0; j < 32; ++j, q += step, gate += gstep) {
 					const float x = v[j] + bias;
 					if (j >= left || !live) continue;
 					if constexpr (E == EPI_F32) {
 						if (aside) *(bf16*)q = __float2bfloat16_rn(x);
 						else *(float*)q = x;
 					} else if constexpr (E == EPI_ACT) *(bf16*)q = __float2bfloat16_rn(x);
+					else if constexpr (E == TG_ACT_GATE) *(bf16*)q = __float2bfloat16_rn(x * sigmoidf_(*gate));
 					else {
 						const bf16 h = __float2bfloat16_rn(x);
 						bf16* d = (bf16*)q;
@@ -93,7 +97,8 @@ __device__ __forceinline__ void tg_epilogue(const GemmArgs& a, int z, const Gemm
 }
 // which instance serves a product
 static inline int tg_kind(const GemmArgs& a) {
-	const bool plain = a.out_scale == 0.f && !a.rs && !a.gate && (a.split == 0 || (a.epi == EPI_F32 && a.split_act == 1));
+	const bool plain = a.out_scale == 0.f && a.out_cap == 0.f && !a.rs && (a.split == 0 || (a.epi == EPI_F32 && a.split_act == 1));
+	if (a.gate) return plain && a.epi == EPI_ACT ? TG_ACT_GATE : TG_ANY;
 	return plain && (a.epi == EPI_F32 || a.epi == EPI_ACT || a.epi == EPI_SPLIT3 || a.epi == EPI_GLU) ? a.epi : TG_ANY;
 }
 
@@ -204,7 +209,7 @@ static inline void gemm_tc_setup() {
 	CUDA_CHECK(cudaHostAlloc((void**)&g_tg.err_host, sizeof(int), cudaHostAllocMapped));
 	*g_tg.err_host = 0;
 	CUDA_CHECK(cudaHostGetDevicePointer((void**)&g_tg.err_dev, g_tg.err_host, 0));
-	for (auto k : {k_seq_gemm_tc<TG_ANY>, k_seq_gemm_tc<EPI_F32>, k_seq_gemm_tc<EPI_ACT>, k_seq_gemm_tc<EPI_SPLIT3>, k_seq_gemm_tc<EPI_GLU>})
+	for (auto k : {k_seq_gemm_tc<TG_ANY>, k_seq_gemm_tc<EPI_F32>, k_seq_gemm_tc<EPI_ACT>, k_seq_gemm_tc<EPI_SPLIT3>, k_seq_gemm_tc<EPI_GLU>, k_seq_gemm_tc<TG_ACT_GATE>})
 		CUDA_CHECK(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, TG_SMEM));
 }
 // a stalled pipeline leaves its code here; read after the stream has been synchronised
@@ -256,6 +261,7 @@ static inline bool gemm_tc_launch(const GemmArgs& a, int batch, cudaStream_t str
 	case EPI_ACT: go(k_seq_gemm_tc<EPI_ACT>); break;
 	case EPI_SPLIT3: go(k_seq_gemm_tc<EPI_SPLIT3>); break;
 	case EPI_GLU: go(k_seq_gemm_tc<EPI_GLU>); break;
+	case TG_ACT_GATE: go(k_seq_gemm_tc<TG_ACT_GATE>); break;
 	default: go(k_seq_gemm_tc<TG_ANY>);
 	}
 	return true;

@@ -95,25 +95,47 @@ __global__ void k_seq_dyt(AT* out, const float* x, const int* rows, const bf16* 
 	out[i] = to_act<AT>(tanhf(a * x[src]) * ldf(w + c) + ldf(b + c));
 }
 
+// sum over the CTA (whole warps, at most 8 of them); every thread adds the warps' sums in the same order
+__device__ __forceinline__ float cta_sum(float v, float* red) {
+	v = warp_sum(v);
+	if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+	__syncthreads();
+	v = 0.f;
+	for (int i = 0; i < (int)(blockDim.x >> 5); ++i) v += red[i];
+	return v;
+}
 // RMS norm of whole rows: out[r][i] = x[row][i] / sqrt(mean(x[row]^2) + eps) * (w[i] + offset); one CTA per row (a single decoded
 // token of a wide model is one row: a warp alone would walk it in a hundred dependent steps), the row is read once (up to
-// blockDim * RMS_KEEP columns stay in registers, wider rows are read a second time)
+// blockDim * RMS_KEEP columns stay in registers, wider rows are read again).  LN: a layer norm without bias, the row's mean is taken
+// off first and the mean square is that of the deviations.
 #define RMS_KEEP 16
-template <typename AT>
+template <typename AT, bool LN = false>
 __global__ void __launch_bounds__(256) k_seq_rms(AT* out, const float* x, const int* rows, const bf16* w, float offset, float eps, int R, int width) {
 	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
-	__shared__ float red[8];
+	__shared__ float red[8], redm[8];
 	const int tid = threadIdx.x, nt = blockDim.x, r = blockIdx.x;
 	const float* src = x + (size_t)(rows ? rows[r] : r) * width;
 	float keep[RMS_KEEP];
-	float ss = 0.f;
+	float ss = 0.f, mean = 0.f;
+	if constexpr (LN) {
+		float sum = 0.f;
+#pragma unroll
+		for (int i = 0; i < RMS_KEEP; ++i) {
+			const int c = i * nt + tid;
+			keep[i] = c < width ? src[c] : 0.f;
+			sum += keep[i];
+		}
+		for (int c = RMS_KEEP * nt + tid; c < width; c += nt) sum += src[c];
+		mean = cta_sum(sum, redm) / (float)width;
+	}
 #pragma unroll
 	for (int i = 0; i < RMS_KEEP; ++i) {
 		const int c = i * nt + tid;
-		keep[i] = c < width ? src[c] : 0.f;
+		if constexpr (LN) keep[i] = c < width ? keep[i] - mean : 0.f;
+		else keep[i] = c < width ? src[c] : 0.f;
 		ss = fmaf(keep[i], keep[i], ss);
 	}
-	for (int c = RMS_KEEP * nt + tid; c < width; c += nt) ss = fmaf(src[c], src[c], ss);
+	for (int c = RMS_KEEP * nt + tid; c < width; c += nt) ss = fmaf(src[c] - mean, src[c] - mean, ss);
 	ss = warp_sum(ss);
 	if ((tid & 31) == 0) red[tid >> 5] = ss;
 	__syncthreads();
@@ -126,7 +148,7 @@ __global__ void __launch_bounds__(256) k_seq_rms(AT* out, const float* x, const 
 		const int c = i * nt + tid;
 		if (c < width) d[c] = to_act<AT>(keep[i] * rinv * (ldf(w + c) + offset));
 	}
-	for (int c = RMS_KEEP * nt + tid; c < width; c += nt) d[c] = to_act<AT>(src[c] * rinv * (ldf(w + c) + offset));
+	for (int c = RMS_KEEP * nt + tid; c < width; c += nt) d[c] = to_act<AT>((src[c] - mean) * rinv * (ldf(w + c) + offset));
 }
 
 // RMS norm with a weight over `len` columns of src rows: segment s of blockIdx.y.  Segment 0 goes to an activation
@@ -159,8 +181,8 @@ __global__ void k_seq_latent_norm(const float* proj, int ldp, RmsSeg sq, RmsSeg 
 	float ss = 0.f;
 	for (int i = lane; i < s.len; i += 32) ss += src[i] * src[i];
 	ss = warp_sum(ss);
-	const float r = 1.f / sqrtf(ss / (float)s.len + eps);
-	if (blockIdx.y == 0) {
+	const float r = 1.f / sqrtf(ss / (float)max(s.len, 1) + eps);
+	if (blockIdx.y == 0) { // (len 0: queries without a latent of their own, only the angles are formed)
 		AT* d = cq + (size_t)n * s.len;
 		for (int i = lane; i < s.len; i += 32) d[i] = to_act<AT>(src[i] * r * ldf(s.w + i));
 		for (int i = lane; i < rope.dims / 2; i += 32) cs[(size_t)n * (rope.dims / 2) + i] = rope_angle(rope, sb.tpos[n], i); // for the queries of this layer
@@ -174,17 +196,18 @@ __global__ void k_seq_latent_norm(const float* proj, int ldp, RmsSeg sq, RmsSeg 
 		}
 	}
 }
-// the rotated query channels of every head: q[n][h * ldh + col + d] from src [N][heads * dims], cs [N][dims / 2] the angles k_seq_latent_norm
+// the rotated query channels of every head: q[n][h * ldh + col + d] from src[n * lds + h * dims + d], cs [N][dims / 2] the angles k_seq_latent_norm
 // formed.  qb given: the queries leave in the activation type instead (split3 = 0), or as [hi | hi | lo] rows of split3 columns each (see
 // k_seq_split_q).  One thread per pair.
-__global__ void __launch_bounds__(256) k_seq_rope_heads(float* q, bf16* qb, int split3, const float* src, const float2* cs, int heads, int dims, long ldq, int ldh, int col, int N) {
+__global__ void __launch_bounds__(256) k_seq_rope_heads(float* q, bf16* qb, int split3, const float* src, long lds, const float2* cs, int heads, int dims, long ldq, int ldh, int col, int N) {
 	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
 	const int half = dims / 2;
 	const size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
 	if (e >= (size_t)N * heads * half) return;
 	const size_t n = e / (heads * half);
 	const int h = (int)(e % (heads * half)) / half, i = (int)(e % half);
-	const float2 uv = *(const float2*)(src + 2 * e), r = rope_turn(cs[n * half + i], uv.x, uv.y);
+	const float* p = src + n * lds + (size_t)h * dims + 2 * i;
+	const float2 r = rope_turn(cs[n * half + i], p[0], p[1]);
 	const size_t o = n * ldq + (size_t)h * ldh + col + 2 * i;
 	if (!qb) {
 		q[o] = r.x, q[o + 1] = r.y;
@@ -356,16 +379,21 @@ struct AttArgs {
 	const int* skip;  // [N] or null: 1 = this token's attention is computed by the product path (k_seq_attn_*), the CTA leaves
 	int nsplit;       // CTAs that share one (token, head tile)'s keys; > 1: partial results go to `part`, k_seq_attention_merge finishes
 	float* part;      // [N][heads][nsplit][vd + 2]: unnormalised output, running maximum, denominator
-	const float* qr = nullptr;  // the last `rot` query channels of every head come from here instead, [N][heads * rot], and are turned by the angles in cs
+	const float* qr = nullptr;  // the last `rot` query channels of every head come from here instead, qr[n * ldqr + h * rot + ..], and are turned by the angles in cs
+	long ldqr = 0;
 	const float2* cs = nullptr; // [N][rot / 2]
 	int rot = 0;
 	int split = 0;    // 1: on the product path queries, keys and probabilities travel as bf16 pairs (value + remainder), so scores and weights keep fp32 accuracy
+	float softcap = 0.f; // > 0: score = softcap tanh(score / softcap), after the scale
+	int vshare = 1;      // neighbouring key heads that read one value head
+	int parts = 0;       // 1: results go to `part` whatever nsplit is (k_seq_attn_diff_merge finishes)
 };
+__device__ __forceinline__ float att_cap(float s, float cap) { return cap > 0.f ? cap * tanhf(s / cap) : s; }
 // channel c of the query of (token, head)
 __device__ __forceinline__ float att_query(const AttArgs& a, int n, int h, int c) {
 	const int e = c - (a.kd - a.rot);
 	if (!a.qr || e < 0) return a.q[((size_t)n * a.heads + h) * a.kd + c];
-	const float* p = a.qr + ((size_t)n * a.heads + h) * a.rot + (e & ~1);
+	const float* p = a.qr + (size_t)n * a.ldqr + (size_t)h * a.rot + (e & ~1);
 	const float2 r = rope_turn(a.cs[(size_t)n * (a.rot / 2) + e / 2], p[0], p[1]);
 	return e & 1 ? r.y : r.x;
 }
@@ -375,7 +403,7 @@ __global__ void __launch_bounds__(ATT_THREADS) k_seq_attention(AttArgs a, AT* ou
 	extern __shared__ float sm[];
 	const int n = blockIdx.x, h0 = blockIdx.y * a.tile, R = a.tile;
 	if (a.skip && a.skip[n]) return;
-	const int kvh = h0 / a.group;
+	const int kvh = h0 / a.group, vh = kvh / a.vshare;
 	float* qs = sm;                  // [R][kd]
 	float* sc = qs + ((R * a.kd + 3) & ~3); // [R][ATT_KC], 16-byte aligned
 	float* mrow = sc + R * ATT_KC;   // [R] running maximum
@@ -432,14 +460,14 @@ __global__ void __launch_bounds__(ATT_THREADS) k_seq_attention(AttArgs a, AT* ou
 						for (int u = 0; u < 4; ++u) dd[u] = warp_sum(dd[u]);
 #pragma unroll
 						for (int u = 0; u < 4; ++u)
-							if (r0 + u < R && lane == u) sc[(r0 + u) * ATT_KC + j] = dd[u] * a.scale - (a.slopes ? a.slopes[h0 + r0 + u] * (float)dist[j] : 0.f);
+							if (r0 + u < R && lane == u) sc[(r0 + u) * ATT_KC + j] = att_cap(dd[u] * a.scale, a.softcap) - (a.slopes ? a.slopes[h0 + r0 + u] * (float)dist[j] : 0.f);
 					}
 				} else {
 					for (int r = 0; r < R; ++r) {
 						float d = 0.f;
 						for (int i = lane; i < a.kd; i += 32) d += qs[r * a.kd + i] * kr[i];
 						d = warp_sum(d);
-						if (lane == 0) sc[r * ATT_KC + j] = d * a.scale - (a.slopes ? a.slopes[h0 + r] * (float)dist[j] : 0.f);
+						if (lane == 0) sc[r * ATT_KC + j] = att_cap(d * a.scale, a.softcap) - (a.slopes ? a.slopes[h0 + r] * (float)dist[j] : 0.f);
 					}
 				}
 			} else if (lane == 0) {
@@ -472,7 +500,7 @@ __global__ void __launch_bounds__(ATT_THREADS) k_seq_attention(AttArgs a, AT* ou
 			for (int k = 0; k < ATT_MAXI; ++k) {
 				const int d = tid + k * ATT_THREADS;
 				if (d < a.vd) {
-					const float* vcol = a.vc + (size_t)kvh * a.vd + d;
+					const float* vcol = a.vc + (size_t)vh * a.vd + d;
 					float s = acc[k] * frow[0];
 					for (int j = 0; j < nk; ++j) s = fmaf(sc[j], vcol[rows[j] * a.vld], s);
 					acc[k] = s;
@@ -483,7 +511,7 @@ __global__ void __launch_bounds__(ATT_THREADS) k_seq_attention(AttArgs a, AT* ou
 			for (int c = 0; c < 2; ++c) {
 				const int d = tid + c * ATT_THREADS;
 				if (d < a.vd) {
-					const float* vcol = a.vc + (size_t)kvh * a.vd + d;
+					const float* vcol = a.vc + (size_t)vh * a.vd + d;
 #pragma unroll
 					for (int r = 0; r < 16; ++r)
 						if (r < R) acc[c * 16 + r] *= frow[r];
@@ -507,7 +535,7 @@ __global__ void __launch_bounds__(ATT_THREADS) k_seq_attention(AttArgs a, AT* ou
 	// accumulator k -> (head of the tile, value column)
 	auto head_of = [&](int k) { return wide ? 0 : k % 16; };
 	auto col_of = [&](int k) { return tid + (wide ? k : k / 16) * ATT_THREADS; };
-	if (a.nsplit > 1) {
+	if (a.nsplit > 1 || a.parts) {
 		const int pw = a.vd + 2;
 #pragma unroll
 		for (int k = 0; k < ATT_MAXI; ++k) {
@@ -590,7 +618,7 @@ __global__ void __launch_bounds__(256) k_seq_attn_mma(AttArgs a, bf16* out, SeqB
 	extern __shared__ __align__(16) float sm[];
 	const int n = blockIdx.x, h0 = blockIdx.y * a.tile, R = a.tile;
 	if (a.skip && a.skip[n]) return;
-	const int kvh = h0 / a.group, kd = a.kd, vd = a.vd, kp = (kd + 15) & ~15;
+	const int kvh = h0 / a.group, vh = kvh / a.vshare, kd = a.kd, vd = a.vd, kp = (kd + 15) & ~15;
 	const int ldk = atm_pad(kd), ldv = shared_kv ? ldk : atm_pad(vd), ldq = atm_ldq(kd);
 	const int kbuf = ATM_KC * ldk, vbuf = shared_kv ? 0 : ATM_KC * ldv;
 	float* const Ks = sm;                                   // [2][ATM_KC][ldk]
@@ -615,7 +643,7 @@ __global__ void __launch_bounds__(256) k_seq_attn_mma(AttArgs a, bf16* out, SeqB
 			const int key = c * ATM_KC + j;
 			if (key < total) {
 				const long row = cache_row(sb, slot, key_pos(key));
-				const float *ksrc = a.kc + row * a.kld + (size_t)kvh * kd, *vsrc = a.vc + row * a.vld + (size_t)kvh * vd;
+				const float *ksrc = a.kc + row * a.kld + (size_t)kvh * kd, *vsrc = a.vc + row * a.vld + (size_t)vh * vd;
 				if (vec) {
 					for (int i = 4 * lane; i < kd; i += 128) cp_async16(kb + j * ldk + i, ksrc + i);
 					if (!shared_kv)
@@ -647,7 +675,7 @@ __global__ void __launch_bounds__(256) k_seq_attn_mma(AttArgs a, bf16* out, SeqB
 #pragma unroll 8
 			for (int c = lane; c < kq; c += 32) put(c, qsrc[c]);
 			for (int i = lane; i < (kd - kq) / 2; i += 32) {
-				const float* p = a.qr + ((size_t)n * a.heads + h0 + r) * a.rot + 2 * i;
+				const float* p = a.qr + (size_t)n * a.ldqr + (size_t)(h0 + r) * a.rot + 2 * i;
 				const float2 v = rope_turn(a.cs[(size_t)n * (a.rot / 2) + i], p[0], p[1]);
 				put(kq + 2 * i, v.x), put(kq + 2 * i + 1, v.y);
 			}
@@ -693,7 +721,7 @@ __global__ void __launch_bounds__(256) k_seq_attn_mma(AttArgs a, bf16* out, SeqB
 			const int r = 2 * warp + i, key = c * ATM_KC + lane;
 			float s = -INFINITY;
 			if (key < total) {
-				s = (sc[r * LDS_ + lane] + sc[16 * LDS_ + r * LDS_ + lane]) * a.scale;
+				s = att_cap((sc[r * LDS_ + lane] + sc[16 * LDS_ + r * LDS_ + lane]) * a.scale, a.softcap);
 				if (a.slopes && r < R) s -= a.slopes[h0 + r] * (float)(pos - key_pos(key));
 			}
 			const float mo = mrow[r], mn = fmaxf(mo, warp_max(s)), p = expf(s - mn);
@@ -738,14 +766,14 @@ __global__ void __launch_bounds__(256) k_seq_attn_mma(AttArgs a, bf16* out, SeqB
 			const int r = g + (e >> 1) * 8, d = (warp + 8 * i) * 8 + 2 * t + (e & 1);
 			if (r >= R || d >= vd) continue;
 			const size_t o = (size_t)n * a.heads + h0 + r;
-			if (a.nsplit > 1) a.part[(o * a.nsplit + blockIdx.z) * (vd + 2) + d] = acc[i][e];
+			if (a.nsplit > 1 || a.parts) a.part[(o * a.nsplit + blockIdx.z) * (vd + 2) + d] = acc[i][e];
 			else {
 				float v = acc[i][e] / lrow[r];
 				if (a.gate) v *= sigmoidf_(a.gate[(size_t)n * a.ldg + (size_t)(h0 + r) * a.ghs + (size_t)d * a.ges]);
 				out[o * vd + d] = __float2bfloat16_rn(v);
 			}
 		}
-	if (a.nsplit > 1 && tid < R) {
+	if ((a.nsplit > 1 || a.parts) && tid < R) {
 		float* p = a.part + (((size_t)n * a.heads + h0 + tid) * a.nsplit + blockIdx.z) * (vd + 2) + vd;
 		p[0] = mrow[tid], p[1] = lrow[tid];
 	}
@@ -830,6 +858,7 @@ struct AttSoftmax {
 	const float* gate; // per head: gate[t * ldg + z], already offset to the first token and head, or null (per-channel gates are applied by the caller)
 	int ldg;
 	int split = 0;     // 1: P rows are 2 Cp wide: the probabilities as bf16, then the bf16 of what that rounding left
+	float softcap = 0.f; // > 0: score = softcap tanh(score / softcap), after the scale
 };
 // One CTA per (row, head).  A thread takes pairs of neighbouring columns; the first SMX_KEEP pairs of its row stay in registers, so a row of up
 // to 512 * SMX_KEEP columns is read once.
@@ -853,7 +882,7 @@ __global__ void __launch_bounds__(256) k_seq_attn_softmax(AttSoftmax a) {
 	const float slope = a.slopes ? a.slopes[z] : 0.f;
 	auto score = [&](int j, float s) { // -inf for a column this row does not see
 		if (j > hi || (j < lo && j >= kept)) return -INFINITY;
-		return s * a.scale - (a.slopes ? slope * (float)(qpos - (j < kfb ? j : a.band.k0 + j - kfb)) : 0.f);
+		return att_cap(s * a.scale, a.softcap) - (a.slopes ? slope * (float)(qpos - (j < kfb ? j : a.band.k0 + j - kfb)) : 0.f);
 	};
 	auto pair = [&](int j) { // j is even and Cp a multiple of 8: both columns lie inside the row
 		if (j > hi || (j + 1 < lo && j >= kept)) return make_float2(-INFINITY, -INFINITY); // nothing was computed there
@@ -912,6 +941,96 @@ __global__ void __launch_bounds__(256) k_seq_attn_softmax(AttSoftmax a) {
 		const float2 v = pair(j);
 		put(j, expf(v.x - mx), expf(v.y - mx));
 	}
+}
+
+// ---------------------------------------------------------------- differential attention: two maps of one head
+// Head h of key group g has two maps over the same values; the attention kernels run them as query heads (g * 2 + map) * group + j
+// of 2 x key heads (j: the head's place in its group).  With their outputs a1, a2: o = a1 - lambda a2, o / sqrt(mean(o^2) + eps) * mul.
+struct AttDiff {
+	int heads, group, vd; // of the result: out[n][heads * vd]
+	float lambda, mul, eps;
+	__device__ __forceinline__ int row(int h, int map) const { return (h / group * 2 + map) * group + h % group; } // query head of a map
+};
+#define ADF_KEEP 8 // value columns per lane kept in registers (heads up to 256 wide; wider ones are formed a second time)
+// both maps' outputs as fp32 rows src[n][2 * heads * vd] (the product path): one warp per (token, head).  only: [N] or null, 1 = this token is here
+template <typename AT>
+__global__ void __launch_bounds__(128) k_seq_attn_diff(AttDiff a, const float* src, AT* out, const int* only, int N) {
+	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
+	const long u = (long)blockIdx.x * 4 + (threadIdx.x >> 5);
+	const int lane = threadIdx.x & 31;
+	if (u >= (long)N * a.heads) return;
+	const int n = (int)(u / a.heads), h = (int)(u % a.heads);
+	if (only && !only[n]) return;
+	const float* p = src + (size_t)n * 2 * a.heads * a.vd;
+	const float *p1 = p + (size_t)a.row(h, 0) * a.vd, *p2 = p + (size_t)a.row(h, 1) * a.vd;
+	float keep[ADF_KEEP], ss = 0.f;
+#pragma unroll
+	for (int i = 0; i < ADF_KEEP; ++i) {
+		const int d = i * 32 + lane;
+		keep[i] = d < a.vd ? p1[d] - a.lambda * p2[d] : 0.f;
+		ss = fmaf(keep[i], keep[i], ss);
+	}
+	for (int d = ADF_KEEP * 32 + lane; d < a.vd; d += 32) {
+		const float v = p1[d] - a.lambda * p2[d];
+		ss = fmaf(v, v, ss);
+	}
+	const float f = a.mul / sqrtf(warp_sum(ss) / (float)a.vd + a.eps);
+	AT* o = out + (size_t)u * a.vd;
+#pragma unroll
+	for (int i = 0; i < ADF_KEEP; ++i)
+		if (i * 32 + lane < a.vd) o[i * 32 + lane] = to_act<AT>(keep[i] * f);
+	for (int d = ADF_KEEP * 32 + lane; d < a.vd; d += 32) o[d] = to_act<AT>((p1[d] - a.lambda * p2[d]) * f);
+}
+// the same from the shares that the attention kernels left in t.part (folded in share order, one or more of them): one CTA per (token, head)
+template <typename AT>
+__global__ void __launch_bounds__(128) k_seq_attn_diff_merge(AttArgs t, AttDiff a, AT* out) {
+	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
+	__shared__ float wz[2][ATT_MAXSPLIT], red[2][2][4], rsum[4];
+	const int n = blockIdx.x, h = blockIdx.y, pw = t.vd + 2, z = threadIdx.x, warp = z >> 5;
+	if (t.skip && t.skip[n]) return;
+	const float *p[2], *b = t.part + (size_t)n * t.heads * t.nsplit * pw;
+	float m[2], l[2];
+#pragma unroll
+	for (int k = 0; k < 2; ++k) {
+		p[k] = b + (size_t)a.row(h, k) * t.nsplit * pw;
+		m[k] = z < t.nsplit ? p[k][z * pw + t.vd] : -INFINITY, l[k] = z < t.nsplit ? p[k][z * pw + t.vd + 1] : 0.f;
+		const float mx = warp_max(m[k]);
+		if ((z & 31) == 0) red[0][k][warp] = mx;
+	}
+	__syncthreads();
+#pragma unroll
+	for (int k = 0; k < 2; ++k) {
+		const float mx = fmaxf(fmaxf(red[0][k][0], red[0][k][1]), fmaxf(red[0][k][2], red[0][k][3]));
+		const float w = m[k] != -INFINITY ? expf(m[k] - mx) : 0.f; // a share without keys counts nothing
+		wz[k][z] = w;
+		const float ls = warp_sum(w * l[k]);
+		if ((z & 31) == 0) red[1][k][warp] = ls;
+	}
+	__syncthreads();
+	const float r1 = 1.f / ((red[1][0][0] + red[1][0][1]) + (red[1][0][2] + red[1][0][3]));
+	const float r2 = a.lambda / ((red[1][1][0] + red[1][1][1]) + (red[1][1][2] + red[1][1][3]));
+	auto value = [&](int d) {
+		float v1 = 0.f, v2 = 0.f;
+#pragma unroll 8
+		for (int k = 0; k < t.nsplit; ++k) v1 = fmaf(p[0][(size_t)k * pw + d], wz[0][k], v1), v2 = fmaf(p[1][(size_t)k * pw + d], wz[1][k], v2);
+		return v1 * r1 - v2 * r2;
+	};
+	float keep[2], ss = 0.f; // value columns z and z + 128 stay in registers
+#pragma unroll
+	for (int i = 0; i < 2; ++i) {
+		keep[i] = i * 128 + z < t.vd ? value(i * 128 + z) : 0.f;
+		ss = fmaf(keep[i], keep[i], ss);
+	}
+	for (int d = 256 + z; d < t.vd; d += 128) {
+		const float v = value(d);
+		ss = fmaf(v, v, ss);
+	}
+	const float f = a.mul / sqrtf(cta_sum(ss, rsum) / (float)a.vd + a.eps);
+	AT* o = out + ((size_t)n * a.heads + h) * a.vd;
+#pragma unroll
+	for (int i = 0; i < 2; ++i)
+		if (i * 128 + z < t.vd) o[i * 128 + z] = to_act<AT>(keep[i] * f);
+	for (int d = 256 + z; d < t.vd; d += 128) o[d] = to_act<AT>(value(d) * f);
 }
 
 // ---------------------------------------------------------------- gated delta rule
@@ -1288,13 +1407,18 @@ struct QkArgs {
 	float* vc;          // cache rows [kv_heads*vdim]
 	int v_norm = 0;     // 1: every value head is divided by its root mean square over vdim (eps inside the root, no weight)
 	int per_head = 0;   // 1: the RMS norms run over each head's `dim` channels, qw / kw are [dim] and serve every head
+	int vheads;         // value heads (kv_heads, or fewer when neighbouring key heads share one)
+	int v_from_k = 0;   // 1: the values are the keys as projected, before norm and rotation (the projection has no value columns)
+	int pairs2 = 0;     // 1: rotation turns channels 2i and 2i + 1 together, 0: i and i + rot_dims/2
+	bf16* qb = nullptr; // given: the queries leave in the activation type for the product path instead, as they are (qsplit 0) or as
+	int qsplit = 0;     //        [hi | hi | lo] rows of `dim` columns each per head (see k_seq_split_q)
 };
 __global__ void __launch_bounds__(256) k_seq_qk_rope(QkArgs a, SeqBatch sb) {
 	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
 	extern __shared__ float cs[]; // [rot_dims/2] cos, [rot_dims/2] sin, then (per_head) [heads + kv_heads] reciprocal root mean squares
 	__shared__ float red[2][8];
 	const int n = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-	const int Q = a.heads * a.dim, K = a.kv_heads * a.dim, Vn = a.kv_heads * a.vdim, half = a.rot_dims / 2;
+	const int Q = a.heads * a.dim, K = a.kv_heads * a.dim, Vn = a.vheads * a.vdim, half = a.rot_dims / 2;
 	const float* pr = a.proj + (size_t)n * a.ldp;
 	const int pos = sb.tpos[n];
 	const long row = cache_row(sb, sb.tslot[n], pos);
@@ -1336,17 +1460,25 @@ __global__ void __launch_bounds__(256) k_seq_qk_rope(QkArgs a, SeqBatch sb) {
 		const int wo = a.per_head ? c - d : 0; // a weight shared by the heads is indexed by the channel inside the head
 		float v = src[c] * r * (w ? ldf(w + c - wo) : 1.f);
 		if (d < a.rot_dims) {
-			const int i = d < half ? d : d - half, o = d < half ? c + half : c - half;
+			const bool first = a.pairs2 ? !(d & 1) : d < half; // the pair's first channel?
+			const int i = a.pairs2 ? d >> 1 : first ? d : d - half, o = a.pairs2 ? (first ? c + 1 : c - 1) : first ? c + half : c - half;
 			const float other = src[o] * r * (w ? ldf(w + o - wo) : 1.f);
-			v = d < half ? v * cs[i] - other * cs[half + i] : v * cs[i] + other * cs[half + i];
+			v = first ? v * cs[i] - other * cs[half + i] : v * cs[i] + other * cs[half + i];
 		}
-		if (isq) a.q[(size_t)n * Q + c] = v;
+		if (isq && a.qb) {
+			const bf16 hi = __float2bfloat16_rn(v);
+			if (a.qsplit) {
+				bf16* qd = a.qb + (size_t)n * 3 * Q + 3 * (c - d) + d;
+				qd[0] = hi, qd[a.dim] = hi, qd[2 * a.dim] = __float2bfloat16_rn(v - __bfloat162float(hi));
+			} else a.qb[(size_t)n * Q + c] = hi;
+		} else if (isq) a.q[(size_t)n * Q + c] = v;
 		else kd[c] = v;
 	}
 	float* vd = a.vc + row * Vn;
+	const float* const vp = pr + Q + (a.v_from_k ? 0 : K);
 	if (a.v_norm) { // one warp per value head
-		for (int g = warp; g < a.kv_heads; g += (int)(blockDim.x >> 5)) {
-			const float* src = pr + Q + K + g * a.vdim;
+		for (int g = warp; g < a.vheads; g += (int)(blockDim.x >> 5)) {
+			const float* src = vp + g * a.vdim;
 			float ss = 0.f;
 			for (int i = lane; i < a.vdim; i += 32) ss = fmaf(src[i], src[i], ss);
 			ss = warp_sum(ss);
@@ -1355,7 +1487,7 @@ __global__ void __launch_bounds__(256) k_seq_qk_rope(QkArgs a, SeqBatch sb) {
 		}
 		return;
 	}
-	for (int i = tid; i < Vn; i += blockDim.x) vd[i] = pr[Q + K + i];
+	for (int i = tid; i < Vn; i += blockDim.x) vd[i] = vp[i];
 }
 
 // ---------------------------------------------------------------- routed experts
@@ -1711,7 +1843,7 @@ __global__ void __launch_bounds__(V == 4 ? 512 : 1024) k_seq_hc_write(float* x, 
 		}
 	}
 }
-// Post-norm blocks: x[n] += y / sqrt(mean(y^2) + eps) * (w + offset), where y = base (a sublayer's last product, or null) + the routed
+// Post-norm blocks: x[n] += y / sqrt(mean(y^2) + eps) * (w + offset) (LN: y's mean is taken off it first), where y = base (a sublayer's last product, or null) + the routed
 // experts' sum when `moe.y` is set (choices in order of rank, each times its weight, or times one when moe.wt is null: the weight went
 // in at the expert's input).  The same pass writes the new row of x in the activation type: the input of the sublayer that follows.
 // One CTA per token.  V = 4: width is a multiple of 4 and a thread owns groups of four neighbouring columns (16-byte loads and stores);
@@ -1729,10 +1861,10 @@ __device__ __forceinline__ void pn_store_act(AT* p, const HcVec<V>& r) {
 		for (int e = 0; e < V; ++e) p[e] = to_act<AT>(r.v[e]);
 	}
 }
-template <typename AT, int V>
+template <typename AT, int V, bool LN = false>
 __global__ void __launch_bounds__(256) k_seq_post_norm(float* x, AT* act, const float* base, HcMoe moe, const bf16* w, float offset, float eps, int N, int width) {
 	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
-	__shared__ float red[8];
+	__shared__ float red[8], redm[8];
 	const int tid = threadIdx.x, nt = blockDim.x;
 	const size_t n = blockIdx.x;
 	auto yval = [&](int c) {
@@ -1750,7 +1882,7 @@ __global__ void __launch_bounds__(256) k_seq_post_norm(float* x, AT* act, const 
 		return y;
 	};
 	HcVec<V> keep[PN_KEEP];
-	float ss = 0.f;
+	float ss = 0.f, sum = 0.f, mean = 0.f;
 #pragma unroll
 	for (int i = 0; i < PN_KEEP; ++i) {
 		const int c = (i * nt + tid) * V;
@@ -1760,10 +1892,35 @@ __global__ void __launch_bounds__(256) k_seq_post_norm(float* x, AT* act, const 
 			for (int e = 0; e < V; ++e) keep[i].v[e] = 0.f;
 		}
 #pragma unroll
-		for (int e = 0; e < V; ++e) ss = fmaf(keep[i].v[e], keep[i].v[e], ss);
+		for (int e = 0; e < V; ++e) {
+			if constexpr (LN) sum += keep[i].v[e];
+			else ss = fmaf(keep[i].v[e], keep[i].v[e], ss);
+		}
 	}
+	if constexpr (LN) {
+		for (int c = (PN_KEEP * nt + tid) * V; c < width; c += nt * V) {
+			const HcVec<V> y = yval(c);
+#pragma unroll
+			for (int e = 0; e < V; ++e) sum += y.v[e];
+		}
+		mean = cta_sum(sum, redm) / (float)width;
+#pragma unroll
+		for (int i = 0; i < PN_KEEP; ++i)
+			if ((i * nt + tid) * V < width) {
+#pragma unroll
+				for (int e = 0; e < V; ++e) keep[i].v[e] -= mean, ss = fmaf(keep[i].v[e], keep[i].v[e], ss);
+			}
+	}
+	auto wide = [&](int c) { // columns beyond the registers: formed again
+		HcVec<V> y = yval(c);
+		if constexpr (LN) {
+#pragma unroll
+			for (int e = 0; e < V; ++e) y.v[e] -= mean;
+		}
+		return y;
+	};
 	for (int c = (PN_KEEP * nt + tid) * V; c < width; c += nt * V) {
-		const HcVec<V> y = yval(c);
+		const HcVec<V> y = wide(c);
 #pragma unroll
 		for (int e = 0; e < V; ++e) ss = fmaf(y.v[e], y.v[e], ss);
 	}
@@ -1787,7 +1944,7 @@ __global__ void __launch_bounds__(256) k_seq_post_norm(float* x, AT* act, const 
 		const int c = (i * nt + tid) * V;
 		if (c < width) put(c, keep[i]);
 	}
-	for (int c = (PN_KEEP * nt + tid) * V; c < width; c += nt * V) put(c, yval(c));
+	for (int c = (PN_KEEP * nt + tid) * V; c < width; c += nt * V) put(c, wide(c));
 }
 // Sandwich blocks: what follows a sublayer's last product, in one pass over the row.
 //   y = (base + the routed experts' sum) * sigmoid(gate),  v = x[n] + y / sqrt(mean(y^2) + eps) * (w + offset);
@@ -2197,6 +2354,7 @@ struct GemmArgs {
 	void* Y2;
 	long ldy2;
 	float out_scale = 0.f;   // != 0: the accumulator (after the bias) is multiplied by it
+	float out_cap = 0.f;     // > 0: then out_cap tanh(. / out_cap)
 	const float* rs = nullptr; // a factor per row on the accumulator (after the bias): rs[(rs_idx ? rs_idx[row] : row) * rs_ld], through a sigmoid when rs_act is 1
 	const int* rs_idx = nullptr;
 	long rs_ld = 1;
@@ -2225,6 +2383,7 @@ __device__ __forceinline__ void gemm_store(const GemmArgs& a, int z, const GemmR
 	const size_t o = (size_t)z * a.ybs + (size_t)(gr.base + n) * a.ldy + m;
 	if (a.bias) acc += ldf(a.bias + (size_t)z * a.M + m);
 	if (a.out_scale != 0.f) acc *= a.out_scale;
+	if (a.out_cap > 0.f) acc = a.out_cap * tanhf(acc / a.out_cap);
 	if (a.rs) {
 		const float f = a.rs[(size_t)(a.rs_idx ? a.rs_idx[gr.base + n] : gr.base + n) * a.rs_ld];
 		acc *= a.rs_act ? sigmoidf_(f) : f;

@@ -163,12 +163,19 @@ void launch_k(Seq& s, void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t sm
 	CUDA_CHECK(cudaLaunchKernelEx(&cfg, kernel, KArgs(args)...));
 }
 
+// attention maps per head (SEQ_GQA: 2 for differential attention); latent attention: query columns in front of the latent, gate rows
+int att_maps(const SeqLayer& L) { return L.type == SEQ_GQA && L.maps > 1 ? L.maps : 1; }
+size_t latent_q(const SeqLayer& L) { return L.q_rank > 0 ? L.q_rank : (size_t)L.heads * L.rot_dims; }
+size_t latent_gate(const SeqLayer& L) { return L.no_gate ? 0 : L.gate_channels ? (size_t)L.heads * L.vdim : L.heads; }
+// fp32 columns of the input projection (q_rank 0: the unrotated query rows leave it in the activation type)
+size_t in_rows(const SeqLayer& L);
+size_t in_cols(const SeqLayer& L) { return in_rows(L) - (L.type == SEQ_LATENT && L.q_rank == 0 ? (size_t)L.heads * L.dim : 0); }
 size_t in_rows(const SeqLayer& L) {
 	switch (L.type) {
-	case SEQ_LATENT: return (size_t)L.q_rank + (L.kv_shared ? 0 : L.kv_rank + L.rot_dims) + (L.no_gate ? 0 : L.heads);
+	case SEQ_LATENT: return latent_q(L) + (L.kv_shared ? 0 : L.kv_rank + L.rot_dims) + latent_gate(L) + (L.q_rank > 0 ? 0 : (size_t)L.heads * L.dim);
 	case SEQ_MINGRU: return (size_t)3 * L.dim;
 	case SEQ_DELTA: return (size_t)2 * L.kv_heads * L.dim + (size_t)L.heads * L.vdim + L.heads + L.a_rank + L.g_rank;
-	case SEQ_GQA: return (size_t)L.heads * L.dim + (size_t)L.kv_heads * L.dim + (size_t)L.kv_heads * L.vdim + (L.no_gate ? 0 : L.gate_per_head ? (size_t)L.heads : (size_t)L.heads * L.vdim);
+	case SEQ_GQA: return (size_t)att_maps(L) * (L.heads + L.kv_heads) * L.dim + (L.v_from_k ? 0 : (size_t)L.kv_heads * L.vdim) + (L.no_gate ? 0 : L.gate_per_head ? (size_t)L.heads : (size_t)L.heads * L.vdim);
 	case SEQ_MLSTM: return (size_t)2 * L.heads * L.dim + (size_t)2 * L.heads * L.vdim + 2 * L.heads;
 	case SEQ_HGRN2: return (size_t)2 * L.heads * L.dim + (size_t)L.heads * L.vdim;
 	case SEQ_MAMBA2: return (size_t)2 * L.heads * L.vdim + (size_t)2 * L.kv_heads * L.dim + L.heads;
@@ -179,7 +186,7 @@ size_t in_rows(const SeqLayer& L) {
 }
 // row stride of the input projection's fp32 output: the mixer's rows, and a router's that ride along (rounded to whole float4s)
 int proj_stride(const SeqLayer& L) {
-	if (L.in_tail <= 0) return (int)in_rows(L);
+	if (L.in_tail <= 0) return (int)in_cols(L);
 	return (int)((in_rows(L) + (L.ff_kind == SEQ_FF_MOE ? L.in_tail : 0) + 3) & ~(size_t)3);
 }
 // a pair whose own record carries the stacked input matrix: column of the second mixer's first row, and the row stride of the fp32 product
@@ -258,7 +265,8 @@ void validate_mixer(const Seq& s, int i, const SeqLayer& L, bool inner) {
 				if (L.taps < 1) CALM_FATAL("seq: layer %d: taps must be positive", i);
 			}
 		} else if (L.type == SEQ_LATENT) {
-			if (L.q_rank < 1 || L.kv_rank < 1) CALM_FATAL("seq: layer %d: latent ranks must be positive", i);
+			if (L.q_rank < 0 || L.kv_rank < 1) CALM_FATAL("seq: layer %d: latent ranks must be positive (q_rank 0: queries without a latent)", i);
+			if (L.q_rank == 0 && (inner || L.in_tail)) CALM_FATAL("seq: layer %d: queries without a latent are served outside pairs and without rows that ride along", i);
 			if (L.rot_dims < 0 || L.rot_dims % 2) CALM_FATAL("seq: layer %d: rot_dims must be even", i);
 				if (L.rot_dims > 0 && !(L.rot_base > 0.f)) CALM_FATAL("seq: layer %d: rot_base must be positive", i);
 				if (L.kv_shared) {
@@ -285,6 +293,11 @@ void validate_mixer(const Seq& s, int i, const SeqLayer& L, bool inner) {
 			if (L.rot_dims > 0 && !(L.rot_base > 0.f)) CALM_FATAL("seq: layer %d: rot_base must be positive", i);
 			if ((L.q_norm == nullptr) != (L.k_norm == nullptr)) CALM_FATAL("seq: layer %d: query and key norm come together", i);
 			if (L.keep_first < 0) CALM_FATAL("seq: layer %d: keep_first is negative", i);
+			if (L.maps < 0 || L.maps > 2) CALM_FATAL("seq: layer %d: one or two attention maps", i);
+			if (L.maps == 2 && (!L.no_gate || L.add_one || L.dist_bias || (L.q_norm && !L.qk_per_head))) CALM_FATAL("seq: layer %d: differential attention has no gate, added one or distance penalty, and norms per head", i);
+			if (L.v_from_k && (L.vdim != L.dim || L.maps == 2)) CALM_FATAL("seq: layer %d: values taken from the keys are as wide as they are (vdim = dim, one map)", i);
+			if (L.rot_kind < 0 || L.rot_kind > 1 || (L.rot_kind == 1 && L.rot_factor > 0.f && !(L.rot_high > L.rot_low && L.rot_low > 0.f && L.rot_original > 0.f)))
+				CALM_FATAL("seq: layer %d: rescaling by wavelength needs 0 < rot_low < rot_high and rot_original > 0", i);
 		} else if (L.type == SEQ_GLA) {
 			if (L.dim > 256) CALM_FATAL("seq: layer %d: a gated-linear-attention head holds at most 256 key channels", i);
 			if (L.a_rank < 1) CALM_FATAL("seq: layer %d: the decay rank must be positive", i);
@@ -295,6 +308,9 @@ void validate_mixer(const Seq& s, int i, const SeqLayer& L, bool inner) {
 		if ((L.type != SEQ_GQA && (L.chunk || L.dist_bias || L.add_one || L.v_norm || L.qk_per_head || L.gate_per_head)) || L.chunk < 0)
 			CALM_FATAL("seq: layer %d: chunk, dist_bias, add_one, v_norm, qk_per_head and gate_per_head are options of SEQ_GQA", i);
 		if (L.type != SEQ_GQA && L.type != SEQ_LATENT && (L.no_gate || L.scores_f32)) CALM_FATAL("seq: layer %d: no_gate and scores_f32 are options of SEQ_GQA and SEQ_LATENT", i);
+		if (L.type != SEQ_GQA && (L.maps > 1 || L.v_from_k || L.rot_pairs || L.rot_kind)) CALM_FATAL("seq: layer %d: maps, v_from_k, rot_pairs and rot_kind are options of SEQ_GQA", i);
+		if (L.type != SEQ_LATENT && L.gate_channels) CALM_FATAL("seq: layer %d: gate_channels is an option of SEQ_LATENT", i);
+		if (L.type != SEQ_GQA && L.type != SEQ_LATENT && L.softcap != 0.f) CALM_FATAL("seq: layer %d: softcap is an option of SEQ_GQA and SEQ_LATENT", i);
 		if (L.type != SEQ_LATENT && L.kv_shared) CALM_FATAL("seq: layer %d: kv_shared is an option of SEQ_LATENT", i);
 		(void)m;
 	}
@@ -344,9 +360,9 @@ void validate(const Seq& s) {
 			}
 		}
 	}
-	if (m.norm_kind != SEQ_NORM_DYT && m.norm_kind != SEQ_NORM_RMS) CALM_FATAL("seq: unknown norm kind %d", m.norm_kind);
+	if (m.norm_kind < SEQ_NORM_DYT || m.norm_kind > SEQ_NORM_LN) CALM_FATAL("seq: unknown norm kind %d", m.norm_kind);
 	if (m.block < SEQ_BLOCK_SERIAL || m.block > SEQ_BLOCK_SANDWICH) CALM_FATAL("seq: unknown block form %d", m.block);
-	if (m.block == SEQ_BLOCK_POST && (m.norm_kind != SEQ_NORM_RMS || m.norm_scalar || m.loop_times > 1)) CALM_FATAL("seq: post-norm blocks use the RMS norm with a weight per column, outside looped spans");
+	if (m.block == SEQ_BLOCK_POST && (m.norm_kind == SEQ_NORM_DYT || m.norm_scalar || m.loop_times > 1)) CALM_FATAL("seq: post-norm blocks use the RMS or layer norm with a weight per column, outside looped spans");
 	if (m.block == SEQ_BLOCK_SANDWICH && (m.norm_kind != SEQ_NORM_RMS || m.norm_scalar || m.loop_times > 1)) CALM_FATAL("seq: sandwich blocks use the RMS norm with a weight per column, outside looped spans");
 	if (m.bigram && (m.bigram_buckets < 1 || m.bigram_mul_prev < 0 || m.bigram_mul_cur < 0)) CALM_FATAL("seq: a bigram table needs buckets >= 1 and multipliers >= 0");
 	if (m.block == SEQ_BLOCK_HYPER && m.norm_kind != SEQ_NORM_RMS) CALM_FATAL("seq: hyper blocks use the RMS norm");
@@ -429,6 +445,7 @@ struct GemmExtra {
 	int x_rows = 0;              // grouped product: rows of X / Y over all groups
 	float epi_f = 0.f;           // EPI_DECAY: exponent
 	float out_scale = 0.f;       // != 0: factor on the accumulator
+	float out_cap = 0.f;         // > 0: soft cap behind it
 	int split = 0;               // columns from here on leave in the activation type to Y2: as relu(.)^2, or unchanged when split_act is 1
 	int split_act = 0;
 	void* Y2 = nullptr;
@@ -455,7 +472,7 @@ void gemm(Seq& s, const void* X, long ldx, long xbs, const void* W, long ldw, lo
 	GemmArgs a;
 	const GemmExtra none;
 	if (!ex) ex = &none;
-	a.bias = (const bf16*)ex->bias, a.res = ex->res, a.gate = ex->gate, a.ldgate = ex->ldgate, a.gbs = ex->gbs, a.seg = ex->seg, a.x_rows = ex->x_rows, a.epi_f = ex->epi_f, a.split = ex->split, a.split_act = ex->split_act, a.Y2 = ex->Y2, a.ldy2 = ex->ldy2, a.out_scale = ex->out_scale;
+	a.bias = (const bf16*)ex->bias, a.res = ex->res, a.gate = ex->gate, a.ldgate = ex->ldgate, a.gbs = ex->gbs, a.seg = ex->seg, a.x_rows = ex->x_rows, a.epi_f = ex->epi_f, a.split = ex->split, a.split_act = ex->split_act, a.Y2 = ex->Y2, a.ldy2 = ex->ldy2, a.out_scale = ex->out_scale, a.out_cap = ex->out_cap;
 	a.rs = ex->rs, a.rs_idx = ex->rs_idx, a.rs_ld = ex->rs_ld, a.rs_act = ex->rs_act;
 	a.split3 = ex->split3, a.glu_mode = ex->glu_mode, a.glu_limit = ex->glu_limit, a.x_idx = ex->x_idx, a.x_div = ex->x_div, a.band_mode = ex->band_mode, a.band_cp = ex->band_cp, a.band = ex->band;
 	a.w_immutable = w_immutable;
@@ -503,8 +520,10 @@ void norm(Seq& s, void* out, const float* x, const int* rows, const SeqNorm& nm,
 	const int W = s.m.width;
 	run_kernel(s, KD_NORM, (double)R * W * (4 + act_size(s)), 0, [&] {
 		const int threads = std::min(256, std::max(32, cdiv(W, 4 * 32) * 32)); // about four columns per thread, whole warps
-		if (s.m.exact) launch_k(s, k_seq_rms<float>, R, threads, 0, (float*)out, x, rows, (const bf16*)nm.w, s.m.norm_offset, s.m.eps, R, W);
-		else launch_k(s, k_seq_rms<bf16>, R, threads, 0, (bf16*)out, x, rows, (const bf16*)nm.w, s.m.norm_offset, s.m.eps, R, W);
+		auto go = [&](auto* o, auto kernel) { launch_k(s, kernel, R, threads, 0, o, x, rows, (const bf16*)nm.w, s.m.norm_offset, s.m.eps, R, W); };
+		const bool ln = s.m.norm_kind == SEQ_NORM_LN;
+		if (s.m.exact) go((float*)out, ln ? k_seq_rms<float, true> : k_seq_rms<float, false>);
+		else go((bf16*)out, ln ? k_seq_rms<bf16, true> : k_seq_rms<bf16, false>);
 	});
 }
 void dyt(Seq& s, void* out, const float* x, const int* rows, const SeqNorm& nm, int R) {
@@ -589,8 +608,9 @@ void reserve_attn(Seq& s, size_t kb, size_t vt, size_t sp) {
 	}
 }
 
-// one sequence's new tokens [first, first + count) at positions pos0.., in blocks of queries that keep S within budget
-void attention_products(Seq& s, int kind, const AttArgs& a, bf16* out, const SeqBatch& sb, int slot, int first, int count, int pos0) {
+// one sequence's new tokens [first, first + count) at positions pos0.., in blocks of queries that keep S within budget.  The result goes to `out`, or
+// (a head's maps that a later kernel combines) as fp32 to `full`
+void attention_products(Seq& s, int kind, const AttArgs& a, bf16* out, float* full, const SeqBatch& sb, int slot, int first, int count, int pos0) {
 	const int G = a.heads / a.group;
 	const size_t budget = (size_t)96 << 20; // elements of S per launch
 	for (int t0 = 0; t0 < count;) {
@@ -610,7 +630,7 @@ void attention_products(Seq& s, int kind, const AttArgs& a, bf16* out, const Seq
 		reserve_attn(s, (size_t)C * a.kd * sx, (size_t)a.vd * Cp * px, (size_t)a.group * Tb * Cp * px);
 		for (int kvh = 0; kvh < G; ++kvh) {
 			AttGather g;
-			g.kc = a.kc, g.vc = a.vc, g.kld = a.kld, g.vld = a.vld, g.kcol = kvh * a.kd, g.vcol = kvh * a.vd, g.kd = a.kd, g.vd = a.vd;
+			g.kc = a.kc, g.vc = a.vc, g.kld = a.kld, g.vld = a.vld, g.kcol = kvh * a.kd, g.vcol = kvh / a.vshare * a.vd, g.kd = a.kd, g.vd = a.vd;
 			g.Kb = s.att_kb, g.Vt = s.att_vt, g.slot = slot, g.k0 = k0, g.C = C, g.Cp = Cp, g.kfb = kfb, g.split = a.split;
 			run_kernel(s, kind, (double)C * (a.kd + a.vd) * (4 + 2 * sx), 0, [&] { launch_k(s, k_seq_attn_gather, dim3(cdiv(Cp, 32), 4), 256, 0, g, sb); });
 			const int h0 = kvh * a.group;
@@ -618,7 +638,8 @@ void attention_products(Seq& s, int kind, const AttArgs& a, bf16* out, const Seq
 			const AttBand band{q0, k0, kfb, a.window > 0 ? a.keep_first : 0, a.window, a.chunk};
 			GemmExtra sx_band, gx;
 			sx_band.band_mode = 1, sx_band.band = band;
-			bf16* const o = out + ((size_t)(first + t0) * a.heads + h0) * a.vd;
+			const size_t o = ((size_t)(first + t0) * a.heads + h0) * a.vd;
+			void* const dst = full ? (void*)(full + o) : (void*)(out + o);
 			// value product: only where the tcgen05 kernel takes it are the columns that a tile of rows does not see left out
 			GemmArgs pv;
 			pv.X = s.att_p, pv.ldx = (long)Cp * px, pv.xbs = (long)Tb * Cp * px, pv.W = s.att_vt, pv.ldw = (long)Cp * px, pv.wbs = 0, pv.N = Tb, pv.M = a.vd, pv.K = a.split ? Cp + C : C, pv.seg = nullptr;
@@ -627,21 +648,22 @@ void attention_products(Seq& s, int kind, const AttArgs& a, bf16* out, const Seq
 			if (banded) gx.band_mode = 2, gx.band = band, gx.band_cp = a.split ? Cp : 0;
 			gemm(s, q, (long)a.heads * a.kd * sx, a.kd * sx, s.att_kb, a.kd * sx, 0, s.att_s, Cp, (long)Tb * Cp, Tb, C, a.kd * sx, a.group, EPI_F32, nullptr, kind, false, &sx_band);
 			AttSoftmax sm;
-			sm.S = s.att_s, sm.P = s.att_p, sm.T = Tb, sm.C = C, sm.Cp = Cp, sm.scale = a.scale, sm.band = band, sm.banded = banded, sm.split = a.split;
+			sm.S = s.att_s, sm.P = s.att_p, sm.T = Tb, sm.C = C, sm.Cp = Cp, sm.scale = a.scale, sm.band = band, sm.banded = banded, sm.split = a.split, sm.softcap = a.softcap;
 			sm.slopes = a.slopes ? a.slopes + h0 : nullptr, sm.add_one = a.add_one;
 			const bool head_gate = a.gate && a.ges == 0; // one gate per head scales the probabilities; a gate per channel goes into the value product's epilogue
 			sm.sink = a.sink ? a.sink + h0 : nullptr, sm.gate = head_gate ? a.gate + (size_t)(first + t0) * a.ldg + h0 : nullptr, sm.ldg = a.ldg;
 			if (a.gate && !head_gate) gx.gate = a.gate + (size_t)(first + t0) * a.ldg + (size_t)h0 * a.ghs, gx.ldgate = a.ldg, gx.gbs = a.ghs;
 			run_kernel(s, kind, (double)a.group * Tb * Cp * (4 + 2 * px), 0, [&] { launch_k(s, k_seq_attn_softmax, dim3(Tb, a.group), 256, 0, sm); });
-			gemm(s, s.att_p, pv.ldx, pv.xbs, s.att_vt, pv.ldw, 0, o, (long)a.heads * a.vd, a.vd, Tb, a.vd, pv.K, a.group, EPI_ACT, nullptr, kind, false, &gx);
+			gemm(s, s.att_p, pv.ldx, pv.xbs, s.att_vt, pv.ldw, 0, dst, (long)a.heads * a.vd, a.vd, Tb, a.vd, pv.K, a.group, full ? EPI_F32 : EPI_ACT, nullptr, kind, false, &gx);
 		}
 		t0 += Tb;
 	}
 }
 
-// q_ready: the queries already wait in a3, in the form the product path reads
-void attention(Seq& s, int kind, AttArgs a, void* out, const SeqBatch& sb, double kv_rows, int longest, bool q_ready = false) {
-	a.skip = nullptr;
+// q_ready: the queries already wait in a3, in the form the product path reads.  diff: a.heads are the maps of diff->heads heads, which a last kernel
+// combines: from fp32 rows in `full` where they were computed as products, from the shares of the keys elsewhere
+void attention(Seq& s, int kind, AttArgs a, void* out, const SeqBatch& sb, double kv_rows, int longest, bool q_ready = false, const AttDiff* diff = nullptr, float* full = nullptr) {
+	a.skip = nullptr, a.parts = diff ? 1 : 0;
 	bool rest = true;
 	if (!s.m.exact && s.attn_products && s.n_on_products > 0) {
 		const size_t n = (size_t)sb.N * a.heads * a.kd;
@@ -649,9 +671,12 @@ void attention(Seq& s, int kind, AttArgs a, void* out, const SeqBatch& sb, doubl
 		} else if (a.split) run_kernel(s, KD_ELEMENT, n * 10.0, 0, [&] { launch_k(s, k_seq_split_q, cdiv(n, 256), 256, 0, (bf16*)s.a3, a.q, a.kd, (size_t)sb.N * a.heads); });
 		else run_kernel(s, KD_ELEMENT, n * 6.0, 0, [&] { launch_k(s, k_seq_cast_cols<bf16>, cdiv(n, 256), 256, 0, (bf16*)s.a3, a.q, a.heads * a.kd, 0, a.heads * a.kd, sb.N); });
 		for (int b = 0; b < sb.B; ++b)
-			if (s.hb_count[b] >= kAttnGemmMin) attention_products(s, kind, a, (bf16*)out, sb, s.hb_slot[b], s.hb_start[b], s.hb_count[b], s.hb_pos0[b]);
+			if (s.hb_count[b] >= kAttnGemmMin) attention_products(s, kind, a, (bf16*)out, diff ? full : nullptr, sb, s.hb_slot[b], s.hb_start[b], s.hb_count[b], s.hb_pos0[b]);
 		a.skip = s.d_skip;
 		rest = s.n_on_products < sb.B;
+		if (diff)
+			run_kernel(s, kind, (double)s.tok_on_products * diff->heads * diff->vd * 10, 0,
+			           [&] { launch_k(s, k_seq_attn_diff<bf16>, cdiv((long)sb.N * diff->heads, 4), 128, 0, *diff, full, (bf16*)out, rest ? s.d_skip : nullptr, sb.N); });
 	}
 	if (!rest) return;
 	const int live = a.skip ? std::max(1, sb.N - s.tok_on_products) : sb.N; // tokens served here (the others' CTAs leave at once)
@@ -663,7 +688,7 @@ void attention(Seq& s, int kind, AttArgs a, void* out, const SeqBatch& sb, doubl
 	ensure_part(s, (size_t)sb.N * a.heads * a.nsplit * (a.vd + 2));
 	a.part = s.part;
 	const dim3 grid(sb.N, a.heads / a.tile, a.nsplit);
-	const double bytes = kv_rows * (a.heads / a.group) * (shared_kv ? a.kd : a.kd + a.vd) * 4.0;
+	const double bytes = kv_rows * (a.heads / a.group) * (shared_kv ? a.kd : a.kd + a.vd / (double)a.vshare) * 4.0;
 	const double flops = 2.0 * kv_rows * a.heads * (a.kd + a.vd);
 	run_kernel(s, kind, a.skip ? 0 : bytes, a.skip ? 0 : flops, [&] {
 		auto al4 = [](long v) { return v % 4 == 0; };
@@ -671,7 +696,13 @@ void attention(Seq& s, int kind, AttArgs a, void* out, const SeqBatch& sb, doubl
 		else if (s.m.exact) launch_k(s, k_seq_attention<float>, grid, ATT_THREADS, p.smem, a, (float*)out, sb);
 		else launch_k(s, k_seq_attention<bf16>, grid, ATT_THREADS, p.smem, a, (bf16*)out, sb);
 	});
-	if (a.nsplit > 1)
+	if (diff)
+		run_kernel(s, kind, 0, 0, [&] {
+			const dim3 mg(sb.N, diff->heads);
+			if (s.m.exact) launch_k(s, k_seq_attn_diff_merge<float>, mg, 128, 0, a, *diff, (float*)out);
+			else launch_k(s, k_seq_attn_diff_merge<bf16>, mg, 128, 0, a, *diff, (bf16*)out);
+		});
+	else if (a.nsplit > 1)
 		run_kernel(s, kind, 0, 0, [&] {
 			const dim3 mg(sb.N, a.heads, cdiv(a.vd, 128));
 			if (s.m.exact) launch_k(s, k_seq_attention_merge<float>, mg, 128, 0, a, (float*)out);
@@ -719,9 +750,10 @@ template <typename AT>
 void post_norm(Seq& s, const float* base, const HcMoe& moe, const SeqNorm& nm, int N) {
 	const int W = s.m.width;
 	run_kernel(s, KD_NORM, (double)N * W * (8.0 + (base ? 4 : 0) + (moe.y ? 4.0 * moe.top : 0) + act_size(s)), 0, [&] {
-		if (W % 4 == 0) // a group of four neighbouring columns per thread up to 1024 columns, whole warps
-			launch_k(s, k_seq_post_norm<AT, 4>, N, std::min(256, cdiv(W / 4, 32) * 32), 0, s.x, (AT*)s.hA, base, moe, (const bf16*)nm.w, s.m.norm_offset, s.m.eps, N, W);
-		else launch_k(s, k_seq_post_norm<AT, 1>, N, std::min(256, cdiv(W, 32) * 32), 0, s.x, (AT*)s.hA, base, moe, (const bf16*)nm.w, s.m.norm_offset, s.m.eps, N, W);
+		auto go = [&](auto kernel, int threads) { launch_k(s, kernel, N, threads, 0, s.x, (AT*)s.hA, base, moe, (const bf16*)nm.w, s.m.norm_offset, s.m.eps, N, W); };
+		const bool ln = s.m.norm_kind == SEQ_NORM_LN;
+		if (W % 4 == 0) go(ln ? k_seq_post_norm<AT, 4, true> : k_seq_post_norm<AT, 4, false>, std::min(256, cdiv(W / 4, 32) * 32)); // a group of four neighbouring columns per thread up to 1024 columns, whole warps
+		else go(ln ? k_seq_post_norm<AT, 1, true> : k_seq_post_norm<AT, 1, false>, std::min(256, cdiv(W, 32) * 32));
 	});
 }
 // write the streams from a sublayer's output; with next_in / next_norm also the normed input of the sublayer that follows (into hA)
@@ -786,17 +818,23 @@ void mixer_typed(Seq& s, const SeqLayer& L, RunState& r, const SeqBatch& sb, dou
 		if (L.in_tail > 0 && L.ff_kind == SEQ_FF_RELU2) gx.split = M, gx.Y2 = s.ah, gx.ldy2 = L.ff, M += L.in_tail;
 		if (L.in_tail == 0 && L.type == SEQ_GLA) // the decay's low-rank input (the last rows) leaves the epilogue in the activation type, ready for its second product
 			gx.split = M - L.a_rank, gx.split_act = 1, gx.Y2 = a1, gx.ldy2 = L.a_rank, a1_ready = true;
+		if (L.type == SEQ_LATENT && L.q_rank == 0) // queries without a latent: their unrotated rows (the last ones) leave in the activation type
+			gx.split = M - L.heads * L.dim, gx.split_act = 1, gx.Y2 = a2, gx.ldy2 = (long)L.heads * L.dim;
 		gemm(s, hA, W, 0, L.w_in, W, 0, s.proj, P, 0, N, M, W, 1, EPI_F32, nullptr, -1, true, &gx);
 	}
 	if (L.type == SEQ_LATENT) {
 		const int H = L.heads, D = L.dim, Dv = L.vdim, Rq = L.q_rank, Rk = L.kv_rank, Pr = L.rot_dims, kd = Rk + Pr;
-		RmsSeg sq{0, Rq, (const bf16*)L.dq_norm}, sc{Rq, Rk, (const bf16*)L.dkv_norm};
+		RmsSeg sq{0, Rq, (const bf16*)L.dq_norm}, sc{(int)latent_q(L), Rk, (const bf16*)L.dkv_norm};
 		const auto rt = s.rot.find(&L);
 		const PairRope rope{Pr, rt == s.rot.end() ? nullptr : rt->second.first, rt == s.rot.end() ? 1.f : rt->second.second};
 		const bool own = !L.kv_shared; // a layer that reads another one's cache has only its query latent to norm
+		const int cl = (int)latent_q(L); // first column of the latent
+		const float* qrot = s.f[1];      // rotated query channels of all heads, as projected
+		long ldqr = (long)H * Pr;
 		run_kernel(s, KD_NORM, (double)N * (Rq + (own ? kd : 0)) * 8, 0,
 		           [&] { launch_k(s, k_seq_latent_norm<AT>, dim3(cdiv(N, 4), own ? 2 : 1), 128, 0, proj, P, sq, sc, a1, r.cache_a, rope, s.rope_cs, sb, s.m.eps); });
-		if (Pr > 0) { // one product for both parts of the queries: the rotated channels stay fp32, the others leave in the activation type
+		if (Rq == 0) qrot = proj, ldqr = P; // both parts came with the input projection
+		else if (Pr > 0) { // one product for both parts of the queries: the rotated channels stay fp32, the others leave in the activation type
 			GemmExtra ux;
 			ux.split = H * Pr, ux.split_act = 1, ux.Y2 = a2, ux.ldy2 = (long)H * D;
 			gemm(s, a1, Rq, 0, L.w_uq, Rq, 0, s.f[1], (long)H * Pr, 0, N, H * (Pr + D), Rq, 1, EPI_F32, nullptr, -1, true, &ux);
@@ -809,18 +847,20 @@ void mixer_typed(Seq& s, const SeqLayer& L, RunState& r, const SeqBatch& sb, dou
 		const bool turned = !direct && (s.m.exact || !s.attn_products || s.n_on_products == 0);
 		if (Pr > 0 && !turned)
 			run_kernel(s, KD_QK, (double)N * H * Pr * (direct ? 4 + 2 * (split3 ? 3 : 1) : 8), 0, [&] {
-				launch_k(s, k_seq_rope_heads, cdiv((long)N * H * Pr / 2, 256), 256, 0, s.f[0], direct ? (bf16*)s.a3 : nullptr, split3, s.f[1], s.rope_cs, H, Pr, (long)H * kq, kq, Rk, N);
+				launch_k(s, k_seq_rope_heads, cdiv((long)N * H * Pr / 2, 256), 256, 0, s.f[0], direct ? (bf16*)s.a3 : nullptr, split3, qrot, ldqr, s.rope_cs, H, Pr, (long)H * kq, kq, Rk, N);
 			});
 		GemmExtra qx;
 		qx.split3 = split3;
 		gemm(s, a2, (long)H * D, D, L.w_ukT, D, (long)Rk * D, direct ? s.a3 : (void*)s.f[0], (long)H * kq, kq, N, Rk, D, H, split3 ? EPI_SPLIT3 : direct ? EPI_ACT : EPI_F32, nullptr, -1, true, &qx);
 		AttArgs a;
 		a.q = s.f[0], a.kc = a.vc = r.cache_a, a.kld = a.vld = kd, a.heads = H, a.group = H, a.kd = kd, a.vd = Rk, a.window = L.window;
-		a.scale = L.scale, a.sink = (const bf16*)L.sink, a.gate = L.no_gate ? nullptr : proj + Rq + (own ? kd : 0), a.ldg = P, a.ghs = 1, a.ges = 0, a.keep_first = 0;
-		a.split = L.scores_f32;
-		if (turned && Pr > 0) a.qr = s.f[1], a.cs = s.rope_cs, a.rot = Pr;
+		a.scale = L.scale, a.sink = (const bf16*)L.sink, a.gate = L.no_gate || L.gate_channels ? nullptr : proj + cl + (own ? kd : 0), a.ldg = P, a.ghs = 1, a.ges = 0, a.keep_first = 0;
+		a.split = L.scores_f32, a.softcap = L.softcap;
+		if (turned && Pr > 0) a.qr = qrot, a.ldqr = ldqr, a.cs = s.rope_cs, a.rot = Pr;
 		attention(s, KD_ATTN_LATENT, a, a1, sb, L.window > 0 ? std::min(kv_rows, (double)N * L.window) : kv_rows, longest, direct);
-		gemm(s, a1, (long)H * Rk, Rk, L.w_uv, Rk, (long)Dv * Rk, a2, (long)H * Dv, Dv, N, Dv, Rk, H, EPI_ACT);
+		GemmExtra vx; // a gate per output channel multiplies the up-projected values in the product's epilogue
+		if (L.gate_channels && !L.no_gate) vx.gate = proj + cl + (own ? kd : 0), vx.ldgate = P, vx.gbs = Dv;
+		gemm(s, a1, (long)H * Rk, Rk, L.w_uv, Rk, (long)Dv * Rk, a2, (long)H * Dv, Dv, N, Dv, Rk, H, EPI_ACT, nullptr, -1, true, &vx);
 		out_product<AT>(s, a2, L.w_o, N, H * Dv, oe, L.b_o);
 	} else if (L.type == SEQ_MINGRU) {
 		const int D = L.dim;
@@ -869,23 +909,28 @@ void mixer_typed(Seq& s, const SeqLayer& L, RunState& r, const SeqBatch& sb, dou
 		           [&] { launch_k(s, k_seq_delta_out<AT>, cdiv((long)N * H, 4), 128, 0, a2, s.f[5], s.f[4], H * Dv, (const bf16*)L.out_norm, N, H, Dv, s.m.eps, 0); });
 		out_product<AT>(s, a2, L.w_o, N, H * Dv, oe, L.b_o);
 	} else if (L.type == SEQ_GQA) {
-		const int H = L.heads, G = L.kv_heads, D = L.dim, Dv = L.vdim;
+		const int maps = att_maps(L), H = L.heads * maps, G = L.kv_heads * maps, D = L.dim, Dv = L.vdim, Gv = L.kv_heads; // a map is a query head (a key head) of its own
+		const int Vn = L.v_from_k ? 0 : Gv * Dv;
 		QkArgs qa;
-		qa.proj = proj, qa.ldp = P, qa.heads = H, qa.kv_heads = G, qa.dim = D, qa.vdim = Dv, qa.qw = (const bf16*)L.q_norm, qa.kw = (const bf16*)L.k_norm, qa.eps = s.m.eps;
+		qa.proj = proj, qa.ldp = P, qa.heads = H, qa.kv_heads = G, qa.vheads = Gv, qa.dim = D, qa.vdim = Dv, qa.qw = (const bf16*)L.q_norm, qa.kw = (const bf16*)L.k_norm, qa.eps = s.m.eps;
 		const auto rt = s.rot.find(&L);
 		qa.rot_dims = rt == s.rot.end() ? 0 : L.rot_dims, qa.freq = rt == s.rot.end() ? nullptr : rt->second.first, qa.mag = rt == s.rot.end() ? 1.f : rt->second.second, qa.q = s.f[0], qa.kc = r.cache_a, qa.vc = r.cache_b;
-		qa.v_norm = L.v_norm, qa.per_head = L.qk_per_head;
+		qa.v_norm = L.v_norm, qa.per_head = L.qk_per_head, qa.v_from_k = L.v_from_k, qa.pairs2 = L.rot_pairs;
+		// when all of the step's attention runs as products the queries go straight to the matrix those read: rounded, or as value and remainder
+		const bool direct = !s.m.exact && s.attn_products && s.n_on_products == sb.B;
+		if (direct) qa.qb = (bf16*)s.a3, qa.qsplit = L.scores_f32;
 		const size_t qk_smem = ((size_t)2 * std::max(L.rot_dims / 2, 1) + H + G) * sizeof(float);
-		run_kernel(s, KD_QK, (double)N * (H * D + G * D + G * Dv) * 8, 0, [&] { launch_k(s, k_seq_qk_rope, N, 256, qk_smem, qa, sb); });
+		run_kernel(s, KD_QK, (double)N * ((H + G) * D * 4.0 + Vn * 4.0 + H * D * (direct ? 2.0 * (L.scores_f32 ? 3 : 1) : 4.0) + (G * D + Gv * Dv) * 4.0), 0, [&] { launch_k(s, k_seq_qk_rope, N, 256, qk_smem, qa, sb); });
 		AttArgs a;
-		a.q = s.f[0], a.kc = r.cache_a, a.vc = r.cache_b, a.kld = G * D, a.vld = G * Dv, a.heads = H, a.group = H / G, a.kd = D, a.vd = Dv;
+		a.q = s.f[0], a.kc = r.cache_a, a.vc = r.cache_b, a.kld = G * D, a.vld = Gv * Dv, a.heads = H, a.group = H / G, a.kd = D, a.vd = Dv, a.vshare = maps;
 		a.window = L.window, a.keep_first = L.window > 0 ? L.keep_first : 0, a.scale = L.scale, a.sink = nullptr;
-		a.gate = L.no_gate ? nullptr : proj + H * D + G * D + G * Dv, a.ldg = P, a.ghs = L.gate_per_head ? 1 : Dv, a.ges = L.gate_per_head ? 0 : 1; // a sigmoid gate per output channel (or per head), from the same stacked projection
+		a.gate = L.no_gate ? nullptr : proj + H * D + G * D + Vn, a.ldg = P, a.ghs = L.gate_per_head ? 1 : Dv, a.ges = L.gate_per_head ? 0 : 1; // a sigmoid gate per output channel (or per head), from the same stacked projection
 		a.chunk = L.chunk, a.slopes = L.dist_bias ? r.slopes : nullptr, a.add_one = L.add_one;
 		const int span = attn_span(L);
-		a.split = L.scores_f32;
-		attention(s, KD_ATTN_WINDOW, a, a2, sb, span > 0 ? std::min(kv_rows, (double)N * span) : kv_rows, longest);
-		out_product<AT>(s, a2, L.w_o, N, H * Dv, oe, L.b_o);
+		a.split = L.scores_f32, a.softcap = L.softcap;
+		const AttDiff df{L.heads, H / G, Dv, L.diff_lambda, L.diff_mul, s.m.eps};
+		attention(s, KD_ATTN_WINDOW, a, a2, sb, span > 0 ? std::min(kv_rows, (double)N * span) : kv_rows, longest, direct, maps > 1 ? &df : nullptr, s.f[2]);
+		out_product<AT>(s, a2, L.w_o, N, L.heads * Dv, oe, L.b_o);
 	} else if (L.type == SEQ_PAIR) {
 		// two mixers on the same normed input: the first one's product lands scaled in the destination, the second one's is added scaled
 		if (oe.epi != EPI_F32) CALM_FATAL("seq: a pair writes its sum to a buffer of its own");
@@ -1235,6 +1280,7 @@ void forward(Seq& s, const SeqBatch& sb, int n_want, double kv_rows, int longest
 		else norm(s, s.hW, s.x, s.d_want, m.final_norm, n_want);
 		GemmExtra lx;
 		lx.out_scale = m.logit_scale != 1.f ? m.logit_scale : 0.f; // 0: no factor
+		lx.out_cap = m.logit_cap;
 		gemm(s, s.hW, m.width, 0, m.head, m.width, 0, s.logits, m.vocab, 0, n_want, m.vocab, m.width, 1, EPI_F32, nullptr, -1, true, &lx);
 	}
 }
@@ -1248,9 +1294,9 @@ void forward_decode_graph(Seq& s, const SeqBatch& sb, int n_want, double kv_rows
 		if (L.type != SEQ_LATENT && L.type != SEQ_WINDOW && L.type != SEQ_GQA) return; // recurrent mixers: nothing to share out
 		const bool lat = L.type == SEQ_LATENT;
 		const int group = lat ? L.heads : L.heads / L.kv_heads, kd = lat ? L.kv_rank + L.rot_dims : L.dim, vd = lat ? L.kv_rank : L.vdim;
-		const int ns = attn_plan(s, group, kd, vd, lat, L.heads, sb.N, attn_span(L), longest).nsplit;
+		const int heads = L.heads * att_maps(L), ns = attn_plan(s, group, kd, vd, lat, heads, sb.N, attn_span(L), longest).nsplit;
 		key.push_back(ns);
-		part_need = std::max(part_need, (size_t)sb.N * L.heads * ns * (vd + 2));
+		part_need = std::max(part_need, (size_t)sb.N * heads * ns * (vd + 2));
 	};
 	for (const RunState& r : s.runs) {
 		const SeqLayer& L = s.layers[r.layer];
@@ -1359,7 +1405,7 @@ extern "C" void* calm_b200_seq_prepare(const struct SeqModel* model) {
 			r.delta = (float*)dalloc(r.delta_per_slot * m.max_seqs * sizeof(float));
 		}
 		if (L.type == SEQ_WINDOW || L.type == SEQ_GQA) {
-			r.cache_a = (float*)dalloc(rows * L.kv_heads * L.dim * sizeof(float));
+			r.cache_a = (float*)dalloc(rows * L.kv_heads * att_maps(L) * L.dim * sizeof(float));
 			r.cache_b = (float*)dalloc(rows * L.kv_heads * L.vdim * sizeof(float));
 		}
 		if (L.type == SEQ_GQA && L.dist_bias) { // the penalty per position of distance: 2^(-8 (h+1) / heads)
@@ -1406,7 +1452,17 @@ extern "C" void* calm_b200_seq_prepare(const struct SeqModel* model) {
 		std::vector<double> f(half);
 		float mag = 1.f;
 		for (int j = 0; j < half; ++j) f[j] = pow((double)L.rot_base, -2.0 * j / dims);
-		if (L.rot_factor > 0.f) {
+		if (L.rot_factor > 0.f && L.rot_kind == 1) {
+			// by wavelength: short waves keep their step, long ones turn `factor` times slower, a blend in the waves per original context between
+			for (int j = 0; j < half; ++j) {
+				const double waves = (double)L.rot_original * f[j] / (2.0 * M_PI); // original / wavelength
+				if (waves < L.rot_low) f[j] /= L.rot_factor;
+				else if (waves <= L.rot_high) {
+					const double sm = (waves - L.rot_low) / ((double)L.rot_high - L.rot_low);
+					f[j] = (1.0 - sm) * f[j] / L.rot_factor + sm * f[j];
+				}
+			}
+		} else if (L.rot_factor > 0.f) {
 			// the pair whose wavelength fits `t` times into the original context: pairs below `lo` keep their step, pairs above `hi`
 			// turn `factor` times slower, a linear ramp between
 			auto where = [&](double t) { return dims * log((double)L.rot_original / (2.0 * M_PI * t)) / (2.0 * log((double)L.rot_base)); };
@@ -1436,7 +1492,7 @@ extern "C" void* calm_b200_seq_prepare(const struct SeqModel* model) {
 			if (L.shared_ff > 0) s.w_fsh = std::max(s.w_fsh, (size_t)2 * L.shared_ff + 1 + L.experts + L.ident);
 			s.w_a = std::max(s.w_a, (size_t)L.shared_ff);
 		}
-		if (L.type == SEQ_GQA) s.w_f = std::max(s.w_f, (size_t)L.heads * L.dim), s.w_a = std::max({s.w_a, (size_t)L.heads * L.vdim, (size_t)L.heads * L.dim * (L.scores_f32 ? 3 : 1)}); // a3 holds the queries (as value + remainder pairs when scores keep fp32 accuracy)
+		if (L.type == SEQ_GQA) s.w_f = std::max({s.w_f, (size_t)L.heads * att_maps(L) * L.dim, att_maps(L) > 1 ? (size_t)L.heads * 2 * L.vdim : 0}), s.w_a = std::max({s.w_a, (size_t)L.heads * L.vdim, (size_t)L.heads * att_maps(L) * L.dim * (L.scores_f32 ? 3 : 1)}); // a3 holds the queries (as value + remainder pairs when scores keep fp32 accuracy)
 		if (L.type == SEQ_GLA) s.w_f = std::max({s.w_f, (size_t)L.heads * L.dim, (size_t)L.heads * L.vdim}), s.w_a = std::max({s.w_a, (size_t)L.heads * L.vdim, (size_t)L.a_rank});
 		if (is_lin(L)) {
 			s.w_f = std::max({s.w_f, (size_t)L.heads * L.dim, (size_t)L.heads * lin_vs(L), (size_t)L.kv_heads * L.dim});

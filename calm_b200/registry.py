@@ -17,13 +17,14 @@ def register(architecture: str, loader: Callable) -> None:
 
 
 def _defaults() -> None:
-    from . import bovinex, fasulix, sopepel, vimulorn, zazilix
+    from . import bovinex, fasulix, sopepel, tabisun, vimulorn, zazilix
 
     register(vimulorn.ARCHITECTURE, vimulorn.load)
     register(bovinex.ARCHITECTURE, bovinex.load)
     register(zazilix.ARCHITECTURE, zazilix.load)
     register(sopepel.ARCHITECTURE, sopepel.load)
     register(fasulix.ARCHITECTURE, fasulix.load)
+    register(tabisun.ARCHITECTURE, tabisun.load)
 
 
 def architecture_of(path: str) -> str:

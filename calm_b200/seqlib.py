@@ -12,7 +12,7 @@ import numpy as np
 
 HERE = os.path.dirname(os.path.abspath(__file__))
 SEQ_LATENT, SEQ_DELTA, SEQ_WINDOW, SEQ_GQA, SEQ_GLA, SEQ_MLSTM, SEQ_HGRN2, SEQ_MAMBA2, SEQ_PAIR, SEQ_MINGRU = 0, 1, 2, 3, 4, 5, 6, 7, 8, 9
-NORM_DYT, NORM_RMS = 0, 1
+NORM_DYT, NORM_RMS, NORM_LN = 0, 1, 2
 BLOCK_SERIAL, BLOCK_PARALLEL, BLOCK_HYPER, BLOCK_POST, BLOCK_SANDWICH = 0, 1, 2, 3, 4
 FF_CLAMPED, FF_RELU2, FF_MOE, FF_GATED = 0, 1, 2, 3
 ACT_SILU, ACT_GELU_TANH = 0, 1
@@ -46,7 +46,9 @@ SeqLayer._fields_ = [(n, C.c_int) for n in ("type", "heads", "kv_heads", "dim", 
                                                                          ("w_sh_gate_up", C.c_void_p), ("w_sh_down", C.c_void_p),
                                                                          ("qk_per_head", C.c_int), ("gate_per_head", C.c_int), ("b_o", C.c_void_p), ("scores_f32", C.c_int), ("ff_act", C.c_int),
                                                                          ("expert_act", C.c_int), ("weight_input", C.c_int), ("shared_gate", C.c_int), ("kv_shared", C.c_int),
-                                                                         ("dwa", C.c_void_p), ("w_rg2", C.c_void_p), ("b_rg2", C.c_void_p)] + [("glu_rows", C.c_int)]
+                                                                         ("dwa", C.c_void_p), ("w_rg2", C.c_void_p), ("b_rg2", C.c_void_p)] + [("glu_rows", C.c_int)] + \
+               [("maps", C.c_int), ("diff_lambda", C.c_float), ("diff_mul", C.c_float), ("v_from_k", C.c_int), ("softcap", C.c_float), ("rot_pairs", C.c_int),
+                ("rot_kind", C.c_int), ("rot_low", C.c_float), ("rot_high", C.c_float), ("gate_channels", C.c_int)]
 
 
 class SeqModel(C.Structure):
@@ -55,7 +57,7 @@ class SeqModel(C.Structure):
                [("embed", C.c_void_p), ("head", C.c_void_p), ("final_norm", SeqNorm), ("layers", C.POINTER(SeqLayer)),
                 ("norm_kind", C.c_int), ("norm_offset", C.c_float), ("block", C.c_int), ("embed_scale", C.c_float),
                 ("streams", C.c_int), ("norm_scalar", C.c_int), ("pos_table", C.c_void_p), ("max_positions", C.c_int),
-                ("bigram", C.c_void_p), ("bigram_buckets", C.c_int), ("bigram_mul_prev", C.c_int), ("bigram_mul_cur", C.c_int), ("logit_scale", C.c_float), ("res_gate", C.c_int)]
+                ("bigram", C.c_void_p), ("bigram_buckets", C.c_int), ("bigram_mul_prev", C.c_int), ("bigram_mul_cur", C.c_int), ("logit_scale", C.c_float), ("res_gate", C.c_int), ("logit_cap", C.c_float)]
 
 
 _lib = None
@@ -101,7 +103,7 @@ class SeqError(RuntimeError):
 
 class SeqDeviceModel:
     """A layer-list model on the GPU.  `layers` are dicts of SeqLayer fields whose tensor-valued entries name tensors in
-    `tensors` (host torch tensors, uploaded here); vimulorn.py, bovinex.py, zazilix.py, sopepel.py and fasulix.py are the hosts that fill them from a checkpoint."""
+    `tensors` (host torch tensors, uploaded here); vimulorn.py, bovinex.py, zazilix.py, sopepel.py, fasulix.py and tabisun.py are the hosts that fill them from a checkpoint."""
 
     def __init__(self, head: Dict[str, object], layers: List[Dict[str, object]], tensors: Dict[str, "object"], exact: bool = False,
                  max_tokens: int = 4096, max_seqs: int = 64, page: int = 16):
@@ -117,7 +119,7 @@ class SeqDeviceModel:
                 self._uploaded[name] = self.lib.calm_b200_seq_upload(t.data_ptr(), t.numel() * t.element_size())
             return self._uploaded[name]
 
-        def norm(prefix: str) -> SeqNorm:  # an RMS norm has only its weight
+        def norm(prefix: str) -> SeqNorm:  # an RMS or layer norm has only its weight
             return SeqNorm(ptr(prefix), ptr(prefix + ".b") if prefix + ".b" in tensors else None, ptr(prefix + ".alpha") if prefix + ".alpha" in tensors else None)
 
         self._subs = []  # the records that pairs point at
@@ -155,6 +157,7 @@ class SeqDeviceModel:
         m.bigram, m.bigram_buckets = ptr(head.get("bigram")), int(head.get("bigram_buckets", 0))
         m.bigram_mul_prev, m.bigram_mul_cur = int(head.get("bigram_mul_prev", 0)), int(head.get("bigram_mul_cur", 0))
         m.logit_scale, m.res_gate = float(head.get("logit_scale", 1.0)), int(head.get("res_gate", 0))
+        m.logit_cap = float(head.get("logit_cap", 0.0))
         m.layers = C.cast(self._layers, C.POINTER(SeqLayer))
         self.desc = m
         self.vocab, self.width = m.vocab, m.width

@@ -71,6 +71,17 @@
  * the heads, is cached behind the latent; both turn by the position, channels 2i and 2i + 1 together; `window`, `sink` and `scores_f32` as
  * for the other attentions; `no_gate` -- no gate rows; `kv_shared` -- the layer has no key/value latent of its own and reads the cache of an earlier one.
  * expert_act 2 -- a routed expert is the clamped gated unit (SeqLayer.limit).
+ * SEQ_NORM_LN: layer norm, (x - mean) / sqrt(mean of squared deviations + eps) * (w + norm_offset), no bias (parallel and post-norm blocks).
+ * Options of SEQ_GQA: `maps` 2 -- differential attention: every head has two query maps and every key head two key maps of `dim` channels over
+ * the same values, each with a softmax of its own; o = a1 - diff_lambda a2, divided by its root mean square over vdim (eps inside), times
+ * diff_mul (no gate then); `v_from_k` -- the values are the keys as projected, before norm and rotation (vdim = dim, no value rows in w_in);
+ * `rot_pairs` -- channels 2i and 2i + 1 turn together; `rot_kind` 1 -- frequencies rescaled by wavelength l: kept below
+ * rot_original / rot_high, divided by rot_factor above rot_original / rot_low, blended between.
+ * Attentions over cached keys (SEQ_GQA, SEQ_LATENT): `softcap` -- score <- softcap tanh(score / softcap) after the scale.
+ * Options of SEQ_LATENT: q_rank 0 -- the queries come straight from the layer's input (no query latent, w_uq or dq_norm); `gate_channels` -- one
+ * sigmoid gate per output channel (heads * vdim gate rows), applied to the up-projected values.
+ * SeqModel.logit_cap: logits <- logit_cap tanh(logits / logit_cap), after logit_scale.
+ * Layers that use another layer's tensors are records of their own that bind the same pointers: cache and state belong to the run.
  * Embedding: SeqModel.bigram adds row (previous token * mul_prev + token * mul_cur) mod buckets of a second table (row `buckets`
  * for a sequence's first token); the previous token is kept with the sequence's slot.  SeqModel.logit_scale multiplies the logits.
  */
@@ -85,7 +96,7 @@ extern "C" {
 #endif
 
 enum SeqMixer { SEQ_LATENT = 0, SEQ_DELTA = 1, SEQ_WINDOW = 2, SEQ_GQA = 3, SEQ_GLA = 4, SEQ_MLSTM = 5, SEQ_HGRN2 = 6, SEQ_MAMBA2 = 7, SEQ_PAIR = 8, SEQ_MINGRU = 9 };
-enum SeqNormKind { SEQ_NORM_DYT = 0, SEQ_NORM_RMS = 1 };
+enum SeqNormKind { SEQ_NORM_DYT = 0, SEQ_NORM_RMS = 1, SEQ_NORM_LN = 2 };
 enum SeqBlock { SEQ_BLOCK_SERIAL = 0, SEQ_BLOCK_PARALLEL = 1, SEQ_BLOCK_HYPER = 2, SEQ_BLOCK_POST = 3, SEQ_BLOCK_SANDWICH = 4 };
 enum SeqFfKind { SEQ_FF_CLAMPED = 0, SEQ_FF_RELU2 = 1, SEQ_FF_MOE = 2, SEQ_FF_GATED = 3 };
 enum SeqFfAct { SEQ_ACT_SILU = 0, SEQ_ACT_GELU_TANH = 1 };
@@ -110,7 +121,7 @@ struct SeqLayer {
 	int type;            /* enum SeqMixer */
 	int heads, kv_heads; /* SEQ_LATENT: kv_heads unused */
 	int dim, vdim;       /* per-head query/key width and value width */
-	int q_rank, kv_rank; /* SEQ_LATENT */
+	int q_rank, kv_rank; /* SEQ_LATENT (q_rank 0: queries without a latent) */
 	int taps;            /* SEQ_DELTA / SEQ_WINDOW: convolution taps (1 = none) */
 	int window;          /* SEQ_WINDOW / SEQ_GQA / SEQ_LATENT: positions seen, the current one included; <= 0: unbounded */
 	int a_rank, g_rank;  /* SEQ_DELTA: inner widths of the decay and gate projections */
@@ -118,8 +129,9 @@ struct SeqLayer {
 	float scale;         /* score scale of the attentions */
 	float limit;         /* clamp of the feed-forward */
 	struct SeqNorm norm1, norm1b, norm2, norm2b;
-	/* SEQ_LATENT: rows [dq | dkv | rotated key part | g] (kv_shared: [dq | g]; no_gate: without g);  SEQ_MINGRU: [z | x | g];  SEQ_DELTA: [q | k | v | b | a1 | g1];  SEQ_WINDOW: [q | k | v];
-	 * SEQ_GQA: [q | k | v | g] (no_gate: [q | k | v]);  SEQ_GLA: [q | k | v | g | a1];  SEQ_MLSTM: [q | k | v | g | i | f];
+	/* SEQ_LATENT: rows [dq | dkv | rotated key part | g] (kv_shared: [dq | g]; no_gate: without g), with q_rank 0 [rotated query rows of all heads | dkv |
+	 * rotated key part | g | unrotated query rows of all heads];  SEQ_MINGRU: [z | x | g];  SEQ_DELTA: [q | k | v | b | a1 | g1];  SEQ_WINDOW: [q | k | v];
+	 * SEQ_GQA: [q | k | v | g] (no_gate: [q | k | v]; v_from_k: without v; maps 2: k rows [key head][map], q rows [key head][map][head of its group]);  SEQ_GLA: [q | k | v | g | a1];  SEQ_MLSTM: [q | k | v | g | i | f];
 	 * SEQ_HGRN2: [q | f | v];  SEQ_MAMBA2: [z | x | B | C | dt] */
 	const void* w_in;
 	const void* w_o;       /* (width, heads*vdim) */
@@ -210,6 +222,15 @@ struct SeqLayer {
 	const void* b_rg2;
 	/* gated units */
 	int glu_rows;          /* 1: the rows of w_gate_up alternate gate and up (row 2c gate c, row 2c + 1 up c), the unit is formed in the product's epilogue */
+	/* SEQ_GQA / SEQ_LATENT, further options */
+	int maps;              /* SEQ_GQA: 2: differential attention (0 is read as 1) */
+	float diff_lambda, diff_mul;
+	int v_from_k;          /* SEQ_GQA: 1: values are the projected keys */
+	float softcap;         /* > 0: soft cap of the scores */
+	int rot_pairs;         /* SEQ_GQA: 1: channels 2i and 2i + 1 turn together (SEQ_LATENT always) */
+	int rot_kind;          /* with rot_factor > 0: 0: ramp over the pair index between rot_fast and rot_slow turns (cos and sin rescaled too); 1: by wavelength */
+	float rot_low, rot_high;
+	int gate_channels;     /* SEQ_LATENT: 1: a gate per output channel instead of per head */
 };
 
 struct SeqModel {
@@ -225,7 +246,7 @@ struct SeqModel {
 	struct SeqNorm final_norm;
 	const struct SeqLayer* layers;
 	int norm_kind;      /* enum SeqNormKind */
-	float norm_offset;  /* SEQ_NORM_RMS: added to the stored weight (1 when the checkpoint keeps weights as offsets from one) */
+	float norm_offset;  /* SEQ_NORM_RMS / SEQ_NORM_LN: added to the stored weight (1 when the checkpoint keeps weights as offsets from one) */
 	int block;          /* enum SeqBlock */
 	float embed_scale;  /* factor on the embedding rows (0 is read as 1) */
 	int streams;        /* SEQ_BLOCK_HYPER: copies of the residual stream (0 is read as 1) */
@@ -236,6 +257,7 @@ struct SeqModel {
 	int bigram_buckets, bigram_mul_prev, bigram_mul_cur;
 	float logit_scale;  /* factor on the logits (0 is read as 1) */
 	int res_gate;       /* SEQ_BLOCK_SANDWICH: 1: a sigmoid gate per column on every sublayer's output */
+	float logit_cap;    /* > 0: soft cap of the logits */
 };
 
 /* cudaMalloc + copy, like upload_cuda */
