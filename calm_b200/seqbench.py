@@ -4,7 +4,8 @@ fp16 on the calm engine; Bovinex beside Vimulorn at the same width, depth, head 
 the same runtime (both have windowed grouped-query attention and a recurrent mixer with a [dim x vdim] state per head); Zazilix
 beside Bovinex likewise (both have grouped-query attention with a bounded view, linear recurrences on the same scan kernel and routed experts);
 Sopepel beside Bovinex too (the same two mixers, grouped-query attention and gated linear attention, side by side in every layer with half the heads each);
-Fasulix beside Vimulorn (latent attention, the clamped unit, a norm before and after every sublayer) and Bovinex (routed experts).
+Fasulix beside Vimulorn (latent attention, the clamped unit, a norm before and after every sublayer) and Bovinex (routed experts);
+Tabisun beside Sopepel (post-norm blocks, attention in chunks of positions with normed heads, a gated dense unit) and Fasulix (latent attention with a sink).
 
 Per size: prompt throughput (one prompt of `prompt` tokens as one step), decode throughput for one sequence and for a
 batch, each after warm-up, timed with CUDA events on the library's stream; then one profiled pass that brackets every
@@ -103,6 +104,26 @@ def fasulix_config(z: dict) -> dict:
     return {"architecture": "Fasulix", "layers": layers, "norm": {"eps": 1e-5}, "vocab": z["vocab"], "width": z["width"]}
 
 
+def tabisun_config(z: dict) -> dict:
+    """Blocks of [capped attention over all earlier positions, latent attention, differential attention in chunks of `window` positions], each with
+    the dense unit.  A head is as wide as the twins' (the differential one's two maps together), half of it rotated in the first, a quarter in the
+    second; with two blocks or more the last one uses the first one's tensors in its first layer."""
+    H, G, D = z["heads"], z["kv_heads"], z["dim"]
+    mlp = {"ff": z["ff"], "kind": "dense"}
+    cap = {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5, "softcap": 50.0,
+           "rot": {"dims": D // 2, "base": 1e6, "scaling": {"factor": 8.0, "original": 4096, "low": 1.0, "high": 4.0}}}
+    lat = {"heads": H, "dim": D - D // 4, "rot_dim": D // 4, "vdim": D, "kv_rank": z["kv_rank"], "scale": D ** -0.5,
+           "rot": {"dims": D // 4, "base": 1e6, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    dif = {"heads": H, "kv_heads": G, "dim": D // 2, "vdim": D, "scale": (D // 2) ** -0.5, "diff": 0.5, "mask": {"size": z["window"]}}
+    layers = []
+    for b in range(z["blocks"]):
+        first = {"type": "attention_2", "mixer": cap, "mlp": mlp}
+        if b > 0 and b == z["blocks"] - 1:
+            first["weights_of"] = 0
+        layers += [first, {"type": "latent_attention", "mixer": lat, "mlp": mlp}, {"type": "attention", "mixer": dif, "mlp": mlp}]
+    return {"architecture": "Tabisun", "layers": layers, "norm": {"eps": 1e-5}, "vocab": z["vocab"], "width": z["width"], "logit_softcap": 30.0}
+
+
 def peaks():
     p = os.path.join(ROOT, "MEASURED_PEAKS.json")
     if os.path.exists(p):
@@ -123,11 +144,11 @@ def roofline_table(stats: dict, hbm_gbs: float, tflops: float) -> dict:
 
 
 def bench_family(family: str, name: str, prompt: int, batch: int, steps: int, warmup: int, seed: int = 0) -> list:
-    from . import bovinex, fasulix, sopepel, vimulorn, zazilix
+    from . import bovinex, fasulix, sopepel, tabisun, vimulorn, zazilix
 
     z = SIZES[name]
     mod, cfg = {"bovinex": (bovinex, bovinex_config(z)), "zazilix": (zazilix, zazilix_config(z, prompt + steps + 2 * warmup + 64)),
-                "sopepel": (sopepel, sopepel_config(z)), "fasulix": (fasulix, fasulix_config(z))}.get(family, (vimulorn, vimulorn_config(z)))
+                "sopepel": (sopepel, sopepel_config(z)), "fasulix": (fasulix, fasulix_config(z)), "tabisun": (tabisun, tabisun_config(z))}.get(family, (vimulorn, vimulorn_config(z)))
     hbm, tf, src = peaks()
     t0 = time.time()
     tensors = mod.random_tensors(cfg, seed)
@@ -224,6 +245,8 @@ def main(sizes, prompt=2048, batch=16, steps=32, warmup=8, twin=True, family="vi
             lines += bench_family("vimulorn", name, prompt, batch, steps, warmup)
         if twin and family in ("zazilix", "sopepel", "fasulix"):
             lines += bench_family("bovinex", name, prompt, batch, steps, warmup)
+        if twin and family == "tabisun":
+            lines += bench_family("sopepel", name, prompt, batch, steps, warmup) + bench_family("fasulix", name, prompt, batch, steps, warmup)
         if llama:
             lines += bench_llama_twin(name, prompt, steps, warmup)
         for ln in lines:
