@@ -51,13 +51,15 @@ __device__ __forceinline__ float softplusf_(float z) { return z > 20.f ? z : log
 
 // x[n] = E[tok[n]] * scale (+ P[position of n], a learned position row, not scaled), written to every one of `streams` copies
 // (and a second copy when a looped span re-adds the embedding).  With a bigram table, row (previous token * mul_prev + token * mul_cur)
-// mod buckets of it is added as well; a sequence's first token (tprev < 0) takes row `buckets`, the table's last.
+// mod buckets of it is added as well; a sequence's first token (tprev < 0) takes row `buckets`, the table's last.  act given: the row also
+// leaves in the activation type (post-norm blocks: the first sublayer's input).
 struct EmbedBigram {
 	const bf16* table; // (buckets + 1, width) or null
 	const int* tprev;  // [N] the token before each packed token in its sequence, -1 for a first token
 	int buckets, mul_prev, mul_cur;
 };
-__global__ void k_seq_embed(float* x, float* x0, const bf16* table, const int* tok, int N, int width, float scale, const bf16* pos_table, const int* tpos, int streams, EmbedBigram bg) {
+template <typename AT>
+__global__ void k_seq_embed(float* x, float* x0, AT* act, const bf16* table, const int* tok, int N, int width, float scale, const bf16* pos_table, const int* tpos, int streams, EmbedBigram bg) {
 	pdl_enter(); // programmatic dependent launch: let the next kernel's launch overlap this one, then wait for the previous one
 	const int n = blockIdx.x;
 	const bf16* e = table + (size_t)tok[n] * width;
@@ -74,6 +76,7 @@ __global__ void k_seq_embed(float* x, float* x0, const bf16* table, const int* t
 		if (br) v += ldf(br + i);
 		for (int s = 0; s < streams; ++s) x[((size_t)n * streams + s) * width + i] = v;
 		if (x0) x0[(size_t)n * width + i] = v;
+		if (act) act[(size_t)n * width + i] = to_act<AT>(v);
 	}
 }
 
@@ -1388,7 +1391,7 @@ __global__ void __launch_bounds__(128) k_seq_gla_scan(GlaArgs a, SeqBatch sb) {
 }
 
 // ---------------------------------------------------------------- query / key preparation of grouped-query attention
-// One CTA per token, on the stacked (biased) projection [q | k | v | ...]: an RMS norm over the WHOLE query projection and one over
+// One CTA per token (or, with norms per head, several: gridDim.y slices of the heads), on the stacked (biased) projection [q | k | v | ...]: an RMS norm over the WHOLE query projection and one over
 // the whole key projection (all heads at once, weights qw / kw; null: no norm), then the first rot_dims channels of every head turn
 // by the token's position (channel i with channel i + rot_dims/2, angle = position * freq[i], cos and sin times `mag`); queries go
 // to an activation-independent fp32 matrix, keys and values to their cache rows.  Angles are formed in double: a position in the
@@ -1420,6 +1423,8 @@ __global__ void __launch_bounds__(256) k_seq_qk_rope(QkArgs a, SeqBatch sb) {
 	const int n = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
 	const int Q = a.heads * a.dim, K = a.kv_heads * a.dim, Vn = a.vheads * a.vdim, half = a.rot_dims / 2;
 	const float* pr = a.proj + (size_t)n * a.ldp;
+	const int units = a.heads + a.kv_heads, per = (units + (int)gridDim.y - 1) / (int)gridDim.y; // this CTA's head vectors: query heads, then key heads
+	const int u0 = min(units, (int)blockIdx.y * per), u1 = min(units, u0 + per);
 	const int pos = sb.tpos[n];
 	const long row = cache_row(sb, sb.tslot[n], pos);
 	for (int i = tid; i < half; i += blockDim.x) {
@@ -1430,12 +1435,12 @@ __global__ void __launch_bounds__(256) k_seq_qk_rope(QkArgs a, SeqBatch sb) {
 	float sq = 0.f, sk = 0.f;
 	float* rh = cs + 2 * max(half, 1);
 	if (a.qw && a.per_head) { // one warp per head vector, query heads first: the key heads follow them in the projection
-		for (int u = warp; u < a.heads + a.kv_heads; u += (int)(blockDim.x >> 5)) {
+		for (int u = u0 + warp; u < u1; u += (int)(blockDim.x >> 5)) {
 			const float* src = pr + (size_t)u * a.dim;
 			float ss = 0.f;
 			for (int i = lane; i < a.dim; i += 32) ss = fmaf(src[i], src[i], ss);
 			ss = warp_sum(ss);
-			if (lane == 0) rh[u] = 1.f / sqrtf(ss / (float)a.dim + a.eps);
+			if (lane == 0) rh[u - u0] = 1.f / sqrtf(ss / (float)a.dim + a.eps);
 		}
 	} else if (a.qw) {
 		for (int i = tid; i < Q; i += blockDim.x) sq = fmaf(pr[i], pr[i], sq);
@@ -1451,11 +1456,11 @@ __global__ void __launch_bounds__(256) k_seq_qk_rope(QkArgs a, SeqBatch sb) {
 		rq = 1.f / sqrtf(sq / (float)Q + a.eps), rk = 1.f / sqrtf(sk / (float)K + a.eps);
 	}
 	float* kd = a.kc + row * K;
-	for (int e = tid; e < Q + K; e += blockDim.x) {
+	for (int e = u0 * a.dim + tid; e < u1 * a.dim; e += blockDim.x) {
 		const bool isq = e < Q;
 		const int c = isq ? e : e - Q, d = c % a.dim;
 		const bf16* w = isq ? a.qw : a.kw;
-		const float r = a.per_head && w ? rh[e / a.dim] : isq ? rq : rk; // e / dim: query heads, then key heads
+		const float r = a.per_head && w ? rh[e / a.dim - u0] : isq ? rq : rk; // e / dim: query heads, then key heads
 		const float* src = pr + (isq ? 0 : Q);
 		const int wo = a.per_head ? c - d : 0; // a weight shared by the heads is indexed by the channel inside the head
 		float v = src[c] * r * (w ? ldf(w + c - wo) : 1.f);
@@ -1477,7 +1482,7 @@ __global__ void __launch_bounds__(256) k_seq_qk_rope(QkArgs a, SeqBatch sb) {
 	float* vd = a.vc + row * Vn;
 	const float* const vp = pr + Q + (a.v_from_k ? 0 : K);
 	if (a.v_norm) { // one warp per value head
-		for (int g = warp; g < a.vheads; g += (int)(blockDim.x >> 5)) {
+		for (int g = blockIdx.y * (int)(blockDim.x >> 5) + warp; g < a.vheads; g += (int)(gridDim.y * (blockDim.x >> 5))) {
 			const float* src = vp + g * a.vdim;
 			float ss = 0.f;
 			for (int i = lane; i < a.vdim; i += 32) ss = fmaf(src[i], src[i], ss);
@@ -1487,7 +1492,7 @@ __global__ void __launch_bounds__(256) k_seq_qk_rope(QkArgs a, SeqBatch sb) {
 		}
 		return;
 	}
-	for (int i = tid; i < Vn; i += blockDim.x) vd[i] = vp[i];
+	for (int i = blockIdx.y * blockDim.x + tid; i < Vn; i += gridDim.y * blockDim.x) vd[i] = vp[i];
 }
 
 // ---------------------------------------------------------------- routed experts

@@ -919,8 +919,10 @@ void mixer_typed(Seq& s, const SeqLayer& L, RunState& r, const SeqBatch& sb, dou
 		// when all of the step's attention runs as products the queries go straight to the matrix those read: rounded, or as value and remainder
 		const bool direct = !s.m.exact && s.attn_products && s.n_on_products == sb.B;
 		if (direct) qa.qb = (bf16*)s.a3, qa.qsplit = L.scores_f32;
+		// few tokens: their heads are shared out over several CTAs (a norm over the whole projection keeps them in one)
+		const int slices = L.q_norm && !L.qk_per_head ? 1 : std::max(1, std::min(cdiv(H + G, 8), 2 * s.sms / N));
 		const size_t qk_smem = ((size_t)2 * std::max(L.rot_dims / 2, 1) + H + G) * sizeof(float);
-		run_kernel(s, KD_QK, (double)N * ((H + G) * D * 4.0 + Vn * 4.0 + H * D * (direct ? 2.0 * (L.scores_f32 ? 3 : 1) : 4.0) + (G * D + Gv * Dv) * 4.0), 0, [&] { launch_k(s, k_seq_qk_rope, N, 256, qk_smem, qa, sb); });
+		run_kernel(s, KD_QK, (double)N * ((H + G) * D * 4.0 + Vn * 4.0 + H * D * (direct ? 2.0 * (L.scores_f32 ? 3 : 1) : 4.0) + (G * D + Gv * Dv) * 4.0), 0, [&] { launch_k(s, k_seq_qk_rope, dim3(N, slices), 256, qk_smem, qa, sb); });
 		AttArgs a;
 		a.q = s.f[0], a.kc = r.cache_a, a.vc = r.cache_b, a.kld = G * D, a.vld = Gv * Dv, a.heads = H, a.group = H / G, a.kd = D, a.vd = Dv, a.vshare = maps;
 		a.window = L.window, a.keep_first = L.window > 0 ? L.keep_first : 0, a.scale = L.scale, a.sink = nullptr;
@@ -1184,11 +1186,6 @@ void layer_typed(Seq& s, const SeqLayer& L, RunState& r, const SeqBatch& sb, dou
 	if (s.m.block == SEQ_BLOCK_POST) {
 		// the sublayers read the stream itself: hA holds its rows in the activation type, written by the kernel that last changed them
 		const HcMoe none{nullptr, nullptr, nullptr, nullptr, 0, 0};
-		if (!s.h_ready) {
-			const size_t n = (size_t)N * s.m.width;
-			run_kernel(s, KD_ELEMENT, n * (4.0 + sizeof(AT)), 0, [&] { launch_k(s, k_seq_cast_cols<AT>, cdiv(n, 256), 256, 0, (AT*)s.hA, s.x, s.m.width, 0, s.m.width, N); });
-			s.h_ready = true;
-		}
 		mixer_typed<AT>(s, L, r, sb, kv_rows, longest, OutEpi{EPI_F32, nullptr, s.mo, nullptr});
 		post_norm<AT>(s, s.mo, none, L.norm1, N);
 		if (L.ff > 0) {
@@ -1255,10 +1252,17 @@ void forward(Seq& s, const SeqBatch& sb, int n_want, double kv_rows, int longest
 	const SeqModel& m = s.m;
 	const int N = sb.N;
 	const bool looped = m.loop_times > 1;
+	const bool post = m.block == SEQ_BLOCK_POST; // the first sublayer reads the embedding rows themselves
+	run_kernel(s, KD_EMBED, (double)N * m.width * (2.0 + (m.pos_table ? 2.0 : 0.0) + (m.bigram ? 2.0 : 0.0) + 4.0 * s.streams + (looped || s.depth ? 4.0 : 0.0) + (post ? act_size(s) : 0.0)), 0,
+	           [&] {
+		           auto go = [&](auto* act, auto kernel) {
+			           launch_k(s, kernel, N, 128, 0, s.x, looped ? s.x0 : s.depth ? s.hist : nullptr, act, (const bf16*)m.embed, s.d_tok, N, m.width, m.embed_scale != 0.f ? m.embed_scale : 1.f, (const bf16*)m.pos_table,
+			                    s.d_tpos, s.streams, EmbedBigram{(const bf16*)m.bigram, s.d_tprev, m.bigram_buckets, m.bigram_mul_prev, m.bigram_mul_cur});
+		           };
+		           if (m.exact) go(post ? (float*)s.hA : nullptr, k_seq_embed<float>);
+		           else go(post ? (bf16*)s.hA : nullptr, k_seq_embed<bf16>);
+	           });
 	s.h_ready = false;
-	run_kernel(s, KD_EMBED, (double)N * m.width * (2.0 + (m.pos_table ? 2.0 : 0.0) + (m.bigram ? 2.0 : 0.0) + 4.0 * s.streams + (looped || s.depth ? 4.0 : 0.0)), 0,
-	           [&] { launch_k(s, k_seq_embed, N, 128, 0, s.x, looped ? s.x0 : s.depth ? s.hist : nullptr, (const bf16*)m.embed, s.d_tok, N, m.width, m.embed_scale != 0.f ? m.embed_scale : 1.f, (const bf16*)m.pos_table, s.d_tpos, s.streams,
-	                          EmbedBigram{(const bf16*)m.bigram, s.d_tprev, m.bigram_buckets, m.bigram_mul_prev, m.bigram_mul_cur}); });
 	for (size_t ri = 0; ri < s.runs.size(); ++ri) {
 		RunState& r = s.runs[ri];
 		const SeqLayer& L = s.layers[r.layer];

@@ -107,16 +107,17 @@ def test_registry_finds_the_family(tmp_path):
 
 
 def test_records_match_the_header():
-    """Every field the header adds for this family is in the ctypes mirror, last and in the header's order."""
+    """Every field the header adds for this family is in the ctypes mirror, in the header's order."""
     root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
     text = open(os.path.join(root, "include", "calm_b200_seq.h")).read()
     body = text[text.index("struct SeqLayer {"):text.index("struct SeqModel {")]
     tail = ["glu_rows", "maps", "diff_lambda", "diff_mul", "v_from_k", "softcap", "rot_pairs", "rot_kind", "rot_low", "rot_high", "gate_channels"]
-    assert [n for n, _ in seqlib.SeqLayer._fields_][-len(tail):] == tail
+    names, mnames = [n for n, _ in seqlib.SeqLayer._fields_], [n for n, _ in seqlib.SeqModel._fields_]
+    assert names[names.index(tail[0]):][:len(tail)] == tail
     at = [min(body.index(x) for x in (" " + n + ";", " " + n + ",") if x in body[body.index("glu_rows;") - 1:]) for n in tail]
     assert at == sorted(at)
     model = text[text.index("struct SeqModel {"):]
-    assert [n for n, _ in seqlib.SeqModel._fields_][-2:] == ["res_gate", "logit_cap"] and model.index("res_gate;") < model.index("logit_cap;")
+    assert mnames[mnames.index("res_gate"):][:2] == ["res_gate", "logit_cap"] and model.index("res_gate;") < model.index("logit_cap;")
 
 
 def test_plain_statement_is_causal_and_chunks_bound_the_attention():
